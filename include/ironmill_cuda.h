@@ -101,6 +101,7 @@ int im_cuda_quantize_affine(const void *w_dev, const void *awq_dev, size_t rows,
 typedef struct im_affine_weight im_affine_weight;
 #define IM_DTYPE_F16 0
 #define IM_DTYPE_F32 1
+#define IM_DTYPE_BF16 2
 
 int im_cuda_affine_weight_create(im_device *dev, const void *qdata_host, const void *scales_host,
                                  const void *zeros_host, int param_dtype, const void *awq_f16_host,
@@ -323,6 +324,41 @@ typedef struct im_model_config {
 } im_model_config;
 
 int im_cuda_model_create(im_device *dev, const im_model_config *cfg, im_model **out);
+
+/* Models given as a list of layers (no counterpart in the reference, whose model types are fixed transformer blocks).
+ * A layer adds mixer(n) + ffn(n) to the residual, n = rms_norm(residual) * norm1 (a parallel block); the mixer is one of the
+ * kinds below and ff = 0 leaves the feed-forward out.  Layers loop_start .. loop_stop - 1 run loop_times times in a row with
+ * the same weights and a cache of their own each time; before every such pass the residual becomes
+ * W_in [residual, embedding output] + step[pass].  loop_times = 0: no loop.
+ * Everything after model_create_stack is the ordinary im_model: finalize, prefill, decode, sequences. */
+#define IM_MIXER_LATENT 1   /* latent attention: cached [normed latent | rotated key part], softmax with a sink logit per head */
+#define IM_MIXER_LINEAR 2   /* decayed linear attention: f32 state [dim, vdim] per head, normed and gated output */
+typedef struct im_stack_layer {
+    int mixer, heads, dim, vdim; /* dim: (unrotated) query / key size of a head, vdim: value size */
+    int ff;                      /* feed-forward width, gelu_tanh(gate) * up; 0 = none */
+    /* IM_MIXER_LATENT */
+    int kv_rank, rot_dim, rot_dims; /* latent size; rotated query / key size; how much of it is rotated */
+    float scale;
+    double rot_base;
+    double yarn_factor, yarn_original, yarn_fast, yarn_slow; /* interpolation of long contexts; factor 0 = plain rotation */
+    /* IM_MIXER_LINEAR */
+    const double *decay_host;    /* [heads] */
+} im_stack_layer;
+typedef struct im_stack_config {
+    int vocab, width, num_layers;
+    const im_stack_layer *layers;
+    int loop_start, loop_stop, loop_times;
+    float norm_eps;
+    float logit_softcap;         /* 0 = none */
+    int max_seq_len, max_batch;  /* 0 = 2048 / 1 */
+    int prefill_chunk_size;      /* 0 = the largest */
+    int compute_f32;             /* 0: weights, activations and latent caches in bf16; 1: everything in f32 */
+} im_stack_config;
+int im_cuda_model_create_stack(im_device *dev, const im_stack_config *cfg, im_model **out);
+/* Tensors of such a model under their checkpoint names: embed, embed.norm, loop.in, loop.step, l<i>.norm1,
+ * l<i>.mix.{q,dkv,dkv.norm,uk,uv,sink,o} or l<i>.mix.{q,k,v,g,o,norm}, l<i>.mlp.{gate,up,down}, final.norm, head.
+ * Row-major [out, in]; dtype IM_DTYPE_F16 / F32 / BF16; converted to the compute type (norm weights, sinks, steps: f32). */
+int im_cuda_model_load_tensor(im_model *m, const char *name, const void *data_host, int dtype, int ndim, const int64_t *shape);
 void im_cuda_model_free(im_model *m);
 /* Tensors arrive under their Hugging Face names (crates/ironmill-inference/src/weight_loading.rs:163-426):
  * model.embed_tokens.weight, model.layers.{i}.input_layernorm.weight, .self_attn.{q,k,v,o}_proj.weight,
@@ -365,6 +401,10 @@ int im_cuda_model_decode_greedy(im_model *m, const uint32_t *first_tokens_host, 
  * single-sequence calls above work on slot 0 and the lockstep form of decode_step on slots 0 .. batch - 1:
  * use one interface or the other on a model.  im_cuda_model_reset frees every slot. */
 int im_cuda_model_seq_add(im_model *m, const uint32_t *tokens_host, int n_tokens, int *seq_id_out, float *logits_out_host);
+/* A sequence without tokens yet; and more tokens for a live sequence (a portion of a prompt, of any length), with the
+ * logits of the places want_host[0] < want_host[1] < ... among them: logits_out_host f32 [n_want, vocab]. */
+int im_cuda_model_seq_open(im_model *m, int *seq_id_out);
+int im_cuda_model_seq_extend(im_model *m, int seq_id, const uint32_t *tokens_host, int n_tokens, const int *want_host, int n_want, float *logits_out_host);
 int im_cuda_model_seq_remove(im_model *m, int seq_id);
 int im_cuda_model_seq_position(const im_model *m, int seq_id);   /* tokens in the sequence's cache; -1: no such sequence */
 int im_cuda_model_batch_decode_step(im_model *m, const int *seq_ids, const uint32_t *tokens_host, int n, float *logits_out_host);

@@ -13,6 +13,7 @@ LIB_PATH = os.path.join(HERE, "libironmill_cuda.so")
 IM_OK = 0
 IM_DTYPE_F16 = 0
 IM_DTYPE_F32 = 1
+IM_DTYPE_BF16 = 2
 
 STATUS_NAMES = {
     0: "IM_OK", -1: "IM_ERR_INVALID", -2: "IM_ERR_CUDA", -3: "IM_ERR_ALLOC", -4: "IM_ERR_BOUNDS",
@@ -37,6 +38,14 @@ _SIZE_RESTYPE = ("im_cuda_device_allocated_bytes", "im_cuda_buffer_length", "im_
                  "im_cuda_sdpa_f16_scratch_bytes", "im_cuda_tq_prefill_scratch_bytes")
 _VOID_RESTYPE = ("im_cuda_device_free", "im_cuda_buffer_free", "im_cuda_affine_weight_free", "im_cuda_model_free",
                  "im_cuda_tq_free", "im_cuda_tp_free")
+
+
+def use(path: str) -> None:
+    """Names the library file to load, before the first call (build.ensure() returns it)."""
+    global LIB_PATH
+    if _lib is not None and path != LIB_PATH:
+        raise CudaSysError(-7, f"{LIB_PATH} is already loaded")
+    LIB_PATH = path
 
 
 def lib() -> C.CDLL:

@@ -15,6 +15,16 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 OBJ = os.path.join(HERE, "csrc", "_obj")
 LIB = os.path.join(HERE, "libironmill_cuda.so")
+# A library with one model family only: what a host that serves a single model has to compile.
+FAMILY_SOURCES = {
+    "stack": ("api.cu", "session.cu", "stack.cu", "dense.cu", "latent_attn.cu", "linear_attn.cu"),
+}
+
+
+def family_lib(family: str) -> str:
+    return os.path.join(HERE, f"libironmill_cuda_{family}.so")
+
+
 INCLUDE = os.path.join(os.path.dirname(HERE), "include")
 
 NVCC_FLAGS = [
@@ -42,8 +52,19 @@ def _nccl_include() -> list[str]:
     return []
 
 
-def sources() -> list[str]:
-    return sorted(f for f in os.listdir(CSRC) if f.endswith(".cu"))
+def sources(family: str | None = None) -> list[str]:
+    return sorted(FAMILY_SOURCES[family]) if family else sorted(f for f in os.listdir(CSRC) if f.endswith(".cu"))
+
+
+def _headers() -> list[str]:
+    return [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cuh", ".h"))] + [os.path.join(INCLUDE, f) for f in os.listdir(INCLUDE)]
+
+
+def ensure(family: str) -> str:
+    """The library a model of `family` runs on: the complete one if it is there and current, else the family's own,
+    compiled now if need be."""
+    deps = [os.path.join(CSRC, f) for f in sources()] + _headers()
+    return LIB if not _stale(LIB, deps) else build(family=family)
 
 
 def _stale(target: str, deps: list[str]) -> bool:
@@ -53,13 +74,14 @@ def _stale(target: str, deps: list[str]) -> bool:
     return any(os.path.getmtime(d) > t for d in deps)
 
 
-def build(force: bool = False, verbose: bool = False, ptxas_info: bool = False) -> str:
+def build(force: bool = False, verbose: bool = False, ptxas_info: bool = False, family: str | None = None) -> str:
+    """Compiles what is out of date and links; the complete library, or with `family` that family's."""
     os.makedirs(OBJ, exist_ok=True)
-    headers = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cuh", ".h"))]
-    headers += [os.path.join(INCLUDE, f) for f in os.listdir(INCLUDE)]
+    headers = _headers()
+    lib = family_lib(family) if family else LIB
     nvcc = _nvcc()
     jobs = []
-    for src in sources():
+    for src in sources(family):
         obj = os.path.join(OBJ, src[:-3] + ".o")
         path = os.path.join(CSRC, src)
         if force or _stale(obj, [path] + headers):
@@ -79,14 +101,14 @@ def build(force: bool = False, verbose: bool = False, ptxas_info: bool = False) 
                 sys.stderr.write(f"--- nvcc {src}\n{r.stdout}{r.stderr}")
             if r.returncode != 0:
                 raise RuntimeError(f"nvcc failed on {src}")
-    objs = [os.path.join(OBJ, s[:-3] + ".o") for s in sources()]
-    if force or jobs or _stale(LIB, objs):
-        cmd = [nvcc, "-shared", "-o", LIB, *objs, "-lcudart", "-ldl"]
+    objs = [os.path.join(OBJ, s[:-3] + ".o") for s in sources(family)]
+    if force or jobs or _stale(lib, objs):
+        cmd = [nvcc, "-shared", "-o", lib, *objs, "-lcudart", "-ldl"]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             sys.stderr.write(r.stdout + r.stderr)
             raise RuntimeError("link failed")
-    return LIB
+    return lib
 
 
 if __name__ == "__main__":

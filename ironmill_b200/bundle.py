@@ -12,7 +12,8 @@ from dataclasses import dataclass, field
 
 import numpy as np
 
-_DTYPES = {"float16": np.float16, "float32": np.float32, "uint8": np.uint8, "int8": np.int8, "int32": np.int32}
+# bfloat16 tensors are kept as their 16-bit patterns (numpy has no such type)
+_DTYPES = {"float16": np.float16, "float32": np.float32, "uint8": np.uint8, "int8": np.int8, "int32": np.int32, "bfloat16": np.uint16}
 
 
 class GpuBundleError(Exception):
@@ -181,7 +182,8 @@ class CudaBundleProvider:
         if self.manifest.get("format_version") != 1:
             raise GpuBundleError(f"unsupported format_version {self.manifest.get('format_version')}")
         self.path = path
-        self._config = ModelConfig.from_json(self.manifest.get("model_config"))
+        from .architectures import config_from_json
+        self._config = config_from_json(self.manifest.get("model_config"))
         self._tensors = self.manifest.get("tensors") or {}
 
     def config(self) -> ModelConfig:

@@ -6,8 +6,7 @@
 //   end-of-layer fused kernel), (QK-norm +) RoPE, TurboQuant write of K and V, TurboQuant split
 //   attention + reduce, o_proj, fused residual+RMSNorm, fused gate+up+SiLU, down_proj, fused
 //   residual+RMSNorm+next-layer QKV projection } -> final RMSNorm -> fp16 lm_head.
-// The whole step is captured once per batch size into a CUDA graph; the sequence position lives
-// in device memory so that the graph replays unchanged as the sequence grows.
+// Slots, captured steps and the entry points of a step are the session's (session.cu).
 //
 // Tensor parallelism (not present in the reference): QKV / gate / up are split by output rows
 // (heads), o / down by input columns, KV heads and their caches by rank, lm_head by vocabulary
@@ -17,16 +16,13 @@
 #include <string.h>
 
 #include <algorithm>
-#include <map>
 #include <new>
 #include <string>
 #include <vector>
 
 #include "common.cuh"
 #include "mega.cuh"
-#if defined(__x86_64__)
-#include <immintrin.h>
-#endif
+#include "session.cuh"
 
 #if __has_include(<nccl.h>)
 #include <nccl.h>
@@ -200,9 +196,7 @@ struct Layer {
     float *ks = nullptr, *vs = nullptr, *krn = nullptr;
 };
 
-struct Model {
-    Device *dev = nullptr;
-    im_model_config cfg{};
+struct Model : im_model {
     int nh_l = 0, nkv_l = 0, I_l = 0, vocab_l = 0, world = 1, rank = 0;
     int q_dim = 0, kv_dim = 0, qkv_dim = 0;
     std::vector<Layer> layers;
@@ -212,34 +206,13 @@ struct Model {
     std::vector<float> signs_host, qjl_host;
     __half *cosc = nullptr, *sinc = nullptr;
     // activations, MT = max tokens per forward
-    int MT = 0;
     __half *hidden = nullptr, *norm_out = nullptr, *residual = nullptr, *qkv = nullptr, *q_d = nullptr, *k_d = nullptr,
            *attn_out = nullptr, *ffn_down = nullptr, *ffn_gate = nullptr, *ffn_up = nullptr, *xs_scratch = nullptr, *logits = nullptr,
            *logits_all = nullptr;
     bool gemm_ok = false;  // every projection is INT4 or INT8 group-128: forwards of 16 tokens and more run the tensor-core GEMM
     float *qrot = nullptr;  // [MT, nh_l, 2, hd] rotated queries
-    uint32_t *tokens_dev = nullptr, *tok_hist = nullptr;
-    int *pos_dev = nullptr, *step_dev = nullptr;
-    uint32_t *tokens_pin = nullptr;
-    __half *logits_pin = nullptr;
-    float2 *argmax_cand = nullptr;  // [max_batch][kArgmaxCtas] candidates of the greedy pick
-    unsigned *argmax_counters = nullptr;
-    int *err_pin = nullptr;  // the device's bounded-wait error word, copied back with every step
-    cudaStream_t stream = nullptr;
-    std::map<int, cudaGraphExec_t> graphs;
-    // Cache slots (continuous batching): every sequence owns one of max_batch slots = its rows of every layer's caches
-    // and its position.  The single-sequence calls work on slot 0, the lockstep batch calls on slots 0 .. batch - 1.
-    std::vector<int> slot_pos;      // host copy of the positions
-    std::vector<char> slot_used;    // claimed by im_cuda_model_seq_add
-    int *slot_ident = nullptr;      // device: 0, 1, 2, ... (a one-sequence forward into slot s passes slot_ident + s)
-    int *slot_map = nullptr;        // device: slots of the sequences of the batch being decoded
-    int *slot_pin = nullptr;
-    bool finalized = false;
-    size_t bytes = 0;
-    int launches_per_step = 0;
     float *scratch_ref = nullptr;
     void *pf_dq = nullptr;          // dequantised K' / V' rows of one sequence for prefill chunks (tq_prefill.cu)
-    int prefill_slot_id = -1, prefill_ctx_end = 0;  // set around a prefill chunk's forward: the slot and its positions after the chunk
     float *kv16_scratch = nullptr;  // split partials of the fp16-KV attention (tq_bits == 16)
     size_t kv16_scratch_bytes = 0;
     // whole-token decode kernel (batch 1, single GPU): tables built by mega_prepare()
@@ -249,120 +222,29 @@ struct Model {
     uint2 *mega_phantom_mail = nullptr;
     __half *logits_seq = nullptr;  // [prefill chunk, vocab_l] logits of every token (prefill_all_logits), allocated on first use
     __half *logits_seq_all = nullptr;
-    __half *logits_seq_pin = nullptr;
 #if IM_HAVE_NCCL_H
     ncclComm_t comm = nullptr;
 #endif
     PeerAllreduce xar;
-    std::vector<std::pair<void *, size_t>> allocs;
 
-    int alloc(void **p, size_t n) {
-        int rc = dev_malloc(dev, p, n);
-        if (rc == IM_OK && n) {
-            allocs.push_back({*p, n});
-            bytes += n;
-        }
-        return rc;
-    }
+    ~Model() override;
+    int forward(int nseq, int T, cudaStream_t st, int *launches, Prof *prof, bool all_logits, const int *slots) override;
+    int finalize() override;
+    // the matvec kernels take at most 64 rows per call
+    int prefill_chunk() const override { return gemm_ok ? cfg.prefill_chunk_size : std::min(cfg.prefill_chunk_size, 64); }
+    int alloc_logits_rows() override;
+    void clear_step_error() override;
+    int hidden_rows(int rows, float *out_host) override;
+    size_t step_bytes(int ctx, int batch) const override;
+    const char *family() const override { return "quantized"; }
 };
 
 // Tokens per prefill forward: the tensor-core GEMMs fill the GPU from about a thousand tokens on (a 256-token chunk is
 // 32-112 CTAs per projection), so the default is the largest chunk; the activation buffers are sized for the configured
 // chunk (at most max_seq_len).  prefill_all_logits keeps 256-token chunks: it holds a chunk's logits for every token.
 static const int kPrefillChunk = 2048;
-static const int kAllLogitsChunk = 256;
 static const int kGemmMinTokens = 16;  // from here on the projections are dense contractions: tcgen05 GEMM instead of matvecs
 
-__global__ void advance_pos_kernel(int *pos, const int *slot_map, int n, int by) {
-    pdl_trigger();
-    pdl_wait();
-    if ((int)threadIdx.x < n) pos[slot_map ? slot_map[threadIdx.x] : threadIdx.x] += by;
-}
-__global__ void set_pos_kernel(int *pos, int n, int v) {
-    if ((int)threadIdx.x < n) pos[threadIdx.x] = v;
-}
-
-// Greedy pick per sequence: LAST maximal index (Iterator::max_by keeps the last of equal maxima,
-// crates/ironmill-inference/src/sampling.rs:331-339).  logits are laid out [parts][nseq][vocab_part].
-// grid (kArgmaxCtas, nseq): every CTA scans a slice of the vocabulary and leaves its candidate in `cand`; the last
-// CTA of a sequence to arrive combines the candidates, writes the token and clears the counter for the next launch.
-constexpr int kArgmaxCtas = 64, kArgmaxThreads = 256;
-__device__ __forceinline__ bool argmax_better(float ov, int oi, float best, int bi) {  // is (ov, oi) preferred over (best, bi)?
-    return oi >= 0 && (bi < 0 || ov > best || (ov == best && oi > bi));
-}
-__global__ void __launch_bounds__(kArgmaxThreads) argmax_kernel(const __half *__restrict__ logits, int vocab_part, int parts, int nseq,
-                                                                uint32_t *__restrict__ tokens, uint32_t *__restrict__ hist,
-                                                                const int *__restrict__ step, int hist_stride, int hist_rows,
-                                                                float2 *__restrict__ cand, unsigned *__restrict__ counters) {
-    __shared__ float sv[kArgmaxThreads / 32];
-    __shared__ int si[kArgmaxThreads / 32];
-    __shared__ int s_last;
-    pdl_trigger();
-    pdl_wait();
-    const int seq = blockIdx.y;
-    const int vocab = vocab_part * parts;
-    const int per = (vocab + gridDim.x - 1) / gridDim.x, i0 = blockIdx.x * per, i1 = min(vocab, i0 + per);
-    float best = -INFINITY;
-    int bi = -1;
-    for (int i = i0 + threadIdx.x; i < i1; i += blockDim.x) {
-        const int part = i / vocab_part, j = i % vocab_part;
-        const float v = __half2float(logits[((size_t)part * nseq + seq) * vocab_part + j]);
-        if (!(v < best) || bi < 0) {  // ascending i per thread: ties move to the later index
-            best = v;
-            bi = i;
-        }
-    }
-    auto block_reduce = [&]() {
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-            const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-            if (argmax_better(ov, oi, best, bi)) {
-                best = ov;
-                bi = oi;
-            }
-        }
-        const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-        if (lane == 0) {
-            sv[warp] = best;
-            si[warp] = bi;
-        }
-        __syncthreads();
-        if (threadIdx.x == 0)
-            for (int w = 1; w < (int)(blockDim.x >> 5); w++)
-                if (argmax_better(sv[w], si[w], best, bi)) {
-                    best = sv[w];
-                    bi = si[w];
-                }
-    };
-    block_reduce();
-    if (threadIdx.x == 0) {
-        cand[(size_t)seq * gridDim.x + blockIdx.x] = make_float2(best, __int_as_float(bi));
-        __threadfence();
-        s_last = atomicAdd(&counters[seq], 1u) == gridDim.x - 1;
-    }
-    __syncthreads();
-    if (!s_last) return;
-    __threadfence();
-    best = -INFINITY;
-    bi = -1;
-    if (threadIdx.x < gridDim.x) {
-        const float2 c = __ldcg(&cand[(size_t)seq * gridDim.x + threadIdx.x]);
-        best = c.x;
-        bi = __float_as_int(c.y);
-    }
-    __syncthreads();
-    block_reduce();
-    if (threadIdx.x == 0) {
-        tokens[seq] = (uint32_t)bi;
-        if (hist) hist[(size_t)(*step % hist_rows) * hist_stride + seq] = (uint32_t)bi;
-        counters[seq] = 0;
-    }
-}
-__global__ void bump_kernel(int *step) {
-    pdl_trigger();
-    pdl_wait();
-    *step += 1;
-}
 
 // act[i] = SiLU(gate[i]) * up[i] (crates/ironmill-inference/src/metal/shaders/activation/activation.metal silu_gate), f32 inside
 __global__ void silu_mul_kernel(const __half *__restrict__ gate, const __half *__restrict__ up, __half *__restrict__ out, size_t n) {
@@ -508,29 +390,10 @@ static int tp_allreduce(Model *m, __half *buf, size_t count, cudaStream_t st) {
 #endif
 }
 
-// Per-category GPU timing of one eager step (the counterpart of MetalConfig.kernel_timing /
-// the profile-metal feature, crates/ironmill-inference/src/metal/pipeline.rs:353-422,1215-1234):
-// an event is recorded after each group of launches and the interval is charged to its category.
-enum ProfCat { kCatEmbed = 0, kCatQkv, kCatRope, kCatKvWrite, kCatAttn, kCatOProj, kCatResNorm, kCatFfn, kCatDown, kCatComm, kCatHead, kCatCount };
-struct Prof {
-    cudaStream_t st;
-    std::vector<cudaEvent_t> ev;
-    std::vector<int> cat;
-    void mark(int c) {
-        cudaEvent_t e;
-        cudaEventCreate(&e);
-        cudaEventRecord(e, st);
-        ev.push_back(e);
-        cat.push_back(c);
-    }
-};
-#define IM_MARK(c) do { if (prof) prof->mark(c); } while (0)
 
-#define IM_TRY(expr)                  \
-    do {                              \
-        int _rc = (expr);             \
-        if (_rc != IM_OK) return _rc; \
-    } while (0)
+static int decode_splits(const Model *m, int batch) {
+    return tq_auto_splits(m->dev, batch, 1, m->nkv_l, m->cfg.max_seq_len);
+}
 
 // One forward pass over nseq sequences x T tokens each (decode: T = 1; prefill: nseq = 1).
 // Logits are produced for the last token of every sequence.
@@ -569,9 +432,10 @@ static int attention_block(Model *m, int part, const TqPrep &a, __half *q_buf, L
                                nseq, a.nh, a.nkv, c.max_seq_len, 0, m->pos_dev, T, attn_splits, st, m->qrot, slots);
 }
 
-static int forward(Model *m, int nseq, int T, int attn_splits, cudaStream_t st, int *launches, Prof *prof = nullptr, bool all_logits = false,
-                   const int *slots = nullptr) {
+int Model::forward(int nseq, int T, cudaStream_t st, int *launches, Prof *prof, bool all_logits, const int *slots) {
+    Model *const m = this;
     const im_model_config &c = m->cfg;
+    const int attn_splits = m->prefill_slot_id >= 0 ? tq_auto_splits(m->dev, 1, T, m->nkv_l, m->prefill_ctx_end) : decode_splits(m, nseq);
     const int H = c.hidden_size, hd = c.head_dim, MT = nseq * T;
     const float eps = c.rms_eps;
     const float attn_scale = c.attn_scale != 0.0f ? c.attn_scale : 1.0f / sqrtf((float)hd);
@@ -871,151 +735,65 @@ static int mega_prepare(Model *m) {
     return IM_OK;
 }
 
-static int decode_splits(const Model *m, int batch) {
-    return tq_auto_splits(m->dev, batch, 1, m->nkv_l, m->cfg.max_seq_len);
-}
-
-// mapped: the sequences of the batch live in the slots listed in m->slot_map (continuous batching); otherwise in slots 0 .. batch - 1.
-static int get_graph(Model *m, int batch, cudaGraphExec_t *out, bool mapped = false) {
-    const int key = batch + (mapped ? 1000 : 0);
-    const int *slots = mapped ? m->slot_map : nullptr;
-    auto it = m->graphs.find(key);
-    if (it != m->graphs.end()) {
-        *out = it->second;
-        return IM_OK;
-    }
-    cudaStream_t st = m->stream;
-    // one eager pass first: sets function attributes and warms NCCL outside the capture
-    const int splits = decode_splits(m, batch);
-    IM_TRY(forward(m, batch, 1, splits, st, nullptr, nullptr, false, slots));
-    IM_CUDA_CHECK(cudaStreamSynchronize(st));
-    cudaGraph_t g = nullptr;
-    IM_CUDA_CHECK(cudaStreamBeginCapture(st, cudaStreamCaptureModeThreadLocal));
-    int nl = 0;
-    int rc = forward(m, batch, 1, splits, st, &nl, nullptr, false, slots);
-    if (rc == IM_OK) {
-        const __half *lg = m->world > 1 ? m->logits_all : m->logits;
-        cudaError_t le = launch_k(argmax_kernel, dim3(kArgmaxCtas, batch), dim3(kArgmaxThreads), 0, st, lg, m->vocab_l, m->world, batch, m->tokens_dev,
-                                  m->tok_hist, (const int *)m->step_dev, m->cfg.max_batch, m->cfg.max_seq_len, m->argmax_cand, m->argmax_counters);
-        if (le == cudaSuccess) le = launch_k(bump_kernel, dim3(1), dim3(1), 0, st, m->step_dev);
-        if (le == cudaSuccess) le = launch_k(advance_pos_kernel, dim3(1), dim3(64), 0, st, m->pos_dev, slots, batch, 1);
-        if (le != cudaSuccess) rc = fail(IM_ERR_CUDA, "launch failed: %s", cudaGetErrorString(le));
-        nl += 3;
-    }
-    cudaError_t e = cudaStreamEndCapture(st, &g);
-    if (rc != IM_OK) {
-        if (g) cudaGraphDestroy(g);
-        return rc;
-    }
-    if (e != cudaSuccess) return fail(IM_ERR_CUDA, "graph capture failed: %s", cudaGetErrorString(e));
-    cudaGraphExec_t ge = nullptr;
-    e = cudaGraphInstantiate(&ge, g, 0);
-    cudaGraphDestroy(g);
-    if (e != cudaSuccess) return fail(IM_ERR_CUDA, "graph instantiate failed: %s", cudaGetErrorString(e));
-    m->graphs[key] = ge;
-    m->launches_per_step = nl;
-    *out = ge;
+int Model::alloc_logits_rows() {
+    IM_TRY(alloc((void **)&logits_seq, (size_t)kAllLogitsChunk * vocab_l * 2));
+    if (world > 1) IM_TRY(alloc((void **)&logits_seq_all, (size_t)kAllLogitsChunk * cfg.vocab_size * 2));
+    logits_rows = world > 1 ? logits_seq_all : logits_seq;
     return IM_OK;
 }
 
-// fp16 -> f32 on the host: 128 K logits per step.  With F16C (every x86-64-v3 CPU) eight at a time.
-#if defined(__x86_64__)
-__attribute__((target("avx,f16c"))) static void widen_f16c(const __half *src, float *dst, int n) {
-    int j = 0;
-    for (; j + 8 <= n; j += 8) _mm256_storeu_ps(dst + j, _mm256_cvtph_ps(_mm_loadu_si128(reinterpret_cast<const __m128i *>(src + j))));
-    for (; j < n; j++) dst[j] = __half2float(src[j]);
+void Model::clear_step_error() {
+    if (mega.bar) cudaMemset(mega.bar, 0, (size_t)(7 * cfg.num_layers + 1) * sizeof(unsigned));
 }
+
+int Model::hidden_rows(int rows, float *out_host) {
+    const size_t n = (size_t)rows * cfg.hidden_size;
+    std::vector<__half> tmp(n);
+    IM_CUDA_CHECK(cudaMemcpyAsync(tmp.data(), norm_out, n * sizeof(__half), cudaMemcpyDeviceToHost, stream));
+    IM_CUDA_CHECK(cudaStreamSynchronize(stream));
+    for (size_t i = 0; i < n; i++) out_host[i] = __half2float(tmp[i]);
+    return IM_OK;
+}
+
+size_t Model::step_bytes(int ctx, int batch) const {
+    size_t b = 0;
+    for (const Layer &L : layers) {
+        for (const AffineWeight *w : {L.qkv, L.o, L.gate, L.up, L.down})
+            b += (size_t)w->N * w->K * w->bits / 8 + (size_t)w->N * w->G * 4 + (w->awq ? (size_t)w->K * 2 : 0);
+        b += 2 * (size_t)cfg.hidden_size * 2;
+        b += (size_t)batch * nkv_l * ctx * (2 * cfg.head_dim * cfg.tq_bits / 8 + (cfg.tq_bits == 16 ? 0 : 12));
+    }
+    return b + (size_t)vocab_l * cfg.hidden_size * 2 + (size_t)cfg.hidden_size * 2;
+}
+
+Model::~Model() {
+#if IM_HAVE_NCCL_H
+    for (int p = 0; p < kXarMaxWorld; p++)
+        if (xar.peer[p] && p != rank) cudaIpcCloseMemHandle(xar.peer[p]);
+    if (xar.base) cudaFree(xar.base);
+    if (comm && nccl() && nccl()->CommDestroy) nccl()->CommDestroy(comm);
 #endif
-static void widen(const __half *src, float *dst, int n) {
-#if defined(__x86_64__)
-    static const bool have = __builtin_cpu_supports("f16c") && __builtin_cpu_supports("avx");
-    if (have) return widen_f16c(src, dst, n);
-#endif
-    for (int j = 0; j < n; j++) dst[j] = __half2float(src[j]);
-}
-static void logits_to_host(const Model *m, const __half *pin, int nseq, float *out) {
-    const int vl = m->vocab_l, parts = m->world, V = m->cfg.vocab_size;
-    for (int p = 0; p < parts; p++)
-        for (int s = 0; s < nseq; s++) widen(pin + ((size_t)p * nseq + s) * vl, out + (size_t)s * V + (size_t)p * vl, vl);
+    for (auto &L : layers) {
+        im_cuda_affine_weight_free(static_cast<im_affine_weight *>(L.qkv));
+        im_cuda_affine_weight_free(static_cast<im_affine_weight *>(L.o));
+        im_cuda_affine_weight_free(static_cast<im_affine_weight *>(L.gate));
+        im_cuda_affine_weight_free(static_cast<im_affine_weight *>(L.up));
+        im_cuda_affine_weight_free(static_cast<im_affine_weight *>(L.down));
+    }
+    if (tq) im_cuda_tq_free(tq);
 }
 
-// A kernel whose bounded wait ran out leaves a non-zero word; the step's results are then invalid.  Clears the
-// word and the grid-barrier counters so that the next step starts clean.
-static int step_error_check(Model *m) {
-    if (*m->err_pin == 0) return IM_OK;
-    const int code = *m->err_pin;
-    *m->err_pin = 0;
-    cudaMemset(m->dev->err_flag, 0, sizeof(int));
-    cudaMemset(m->dev->sk_counters, 0, (size_t)kSkMaxBlocks * sizeof(int));
-    if (m->mega.bar) cudaMemset(m->mega.bar, 0, (size_t)(7 * m->cfg.num_layers + 1) * sizeof(unsigned));
-    return fail(IM_ERR_TIMEOUT, "a device-side bounded wait ran out (code %d); the results of this step are invalid", code);
+// The model behind a handle, if it is of this file's family
+static Model *quantized(im_model *h) {
+    Model *m = dynamic_cast<Model *>(h);
+    if (h && !m) fail(IM_ERR_INVALID, "this call is for the quantized Llama / Qwen3 family, the model is of family '%s'", h->family());
+    return m;
 }
-
-// Positions of every slot (reset, truncate of the single-sequence / lockstep interface).
-static int set_positions(Model *m, int pos) {
-    set_pos_kernel<<<1, 64, 0, m->stream>>>(m->pos_dev, m->cfg.max_batch, pos);
-    IM_CUDA_CHECK(cudaGetLastError());
-    for (int &p : m->slot_pos) p = pos;
-    return IM_OK;
-}
-__global__ void set_one_pos_kernel(int *pos, int slot, int v) { pos[slot] = v; }
-
-// Prefill of n tokens into cache slot `slot`, continuing at that slot's position.  last_logits (optional): f32 [vocab]
-// of the last token; all_logits (optional): f32 [n, vocab].
-static int prefill_slot(Model *m, int slot, const uint32_t *tokens_host, int n, float *last_logits, float *all_logits) {
-    if (m->slot_pos[slot] + n > m->cfg.max_seq_len)
-        return fail(IM_ERR_BOUNDS, "sequence position %d + %d tokens exceeds max_seq_len %d", m->slot_pos[slot], n, m->cfg.max_seq_len);
-    cudaStream_t st = m->stream;
-    // 256-token chunks when the projections run as tensor-core GEMMs; the matvec kernels take at most 64 rows per call
-    int chunk = m->gemm_ok ? m->cfg.prefill_chunk_size : (m->cfg.prefill_chunk_size < 64 ? m->cfg.prefill_chunk_size : 64);
-    if (all_logits && chunk > kAllLogitsChunk) chunk = kAllLogitsChunk;
-    const size_t V = (size_t)m->cfg.vocab_size;
-    const int *slots = slot == 0 ? nullptr : m->slot_ident + slot;
-    if (all_logits && !m->logits_seq) {  // first use: a chunk's worth of logits on the device and in pinned host memory
-        IM_TRY(m->alloc((void **)&m->logits_seq, (size_t)kAllLogitsChunk * m->vocab_l * 2));
-        if (m->world > 1) IM_TRY(m->alloc((void **)&m->logits_seq_all, (size_t)kAllLogitsChunk * V * 2));
-        IM_CUDA_CHECK(cudaMallocHost((void **)&m->logits_seq_pin, (size_t)kAllLogitsChunk * V * 2));
-    }
-    for (int done = 0; done < n; done += chunk) {
-        const int T = n - done < chunk ? n - done : chunk;
-        memcpy(m->tokens_pin, tokens_host + done, (size_t)T * 4);
-        IM_CUDA_CHECK(cudaMemcpyAsync(m->tokens_dev, m->tokens_pin, (size_t)T * 4, cudaMemcpyHostToDevice, st));
-        const int splits = tq_auto_splits(m->dev, 1, T, m->nkv_l, m->slot_pos[slot] + T);
-        m->prefill_slot_id = slot;
-        m->prefill_ctx_end = m->slot_pos[slot] + T;
-        const int frc = forward(m, 1, T, splits, st, nullptr, nullptr, all_logits != nullptr, slots);
-        m->prefill_slot_id = -1;
-        IM_TRY(frc);
-        advance_pos_kernel<<<1, 64, 0, st>>>(m->pos_dev, slots, 1, T);
-        IM_CUDA_CHECK(cudaGetLastError());
-        if (all_logits) {
-            const __half *lg = m->world > 1 ? m->logits_seq_all : m->logits_seq;
-            IM_CUDA_CHECK(cudaMemcpyAsync(m->logits_seq_pin, lg, (size_t)T * V * 2, cudaMemcpyDeviceToHost, st));
-        }
-        IM_CUDA_CHECK(cudaMemcpyAsync(m->err_pin, m->dev->err_flag, sizeof(int), cudaMemcpyDeviceToHost, st));
-        IM_CUDA_CHECK(cudaStreamSynchronize(st));  // tokens_pin is reused by the next chunk
-        IM_TRY(step_error_check(m));
-        m->slot_pos[slot] += T;
-        if (all_logits) {  // device layout [part][token][vocab_l] -> host rows [token][vocab]
-            const int vl = m->vocab_l;
-            for (int p = 0; p < m->world; p++)
-                for (int t = 0; t < T; t++)
-                    widen(m->logits_seq_pin + ((size_t)p * T + t) * vl, all_logits + (size_t)(done + t) * V + (size_t)p * vl, vl);
-        }
-    }
-    if (last_logits) {
-        const __half *lg = m->world > 1 ? m->logits_all : m->logits;
-        IM_CUDA_CHECK(cudaMemcpyAsync(m->logits_pin, lg, V * 2, cudaMemcpyDeviceToHost, st));
-        IM_CUDA_CHECK(cudaStreamSynchronize(st));
-        logits_to_host(m, m->logits_pin, 1, last_logits);
-    }
-    return IM_OK;
-}
+static const Model *quantized(const im_model *h) { return dynamic_cast<const Model *>(h); }
 
 }  // namespace im
 
 using namespace im;
-struct im_model : im::Model {};
 
 IM_EXPORT int im_cuda_tp_unique_id(void *id_out_128_bytes) {
     IM_GUARD_BEGIN
@@ -1033,9 +811,11 @@ IM_EXPORT int im_cuda_tp_unique_id(void *id_out_128_bytes) {
     IM_GUARD_END
 }
 
-IM_EXPORT int im_cuda_model_tp_init(im_model *m, const void *id_128_bytes) {
+IM_EXPORT int im_cuda_model_tp_init(im_model *h, const void *id_128_bytes) {
     IM_GUARD_BEGIN
-    IM_REQUIRE(m && id_128_bytes, "bad argument");
+    IM_REQUIRE(h && id_128_bytes, "bad argument");
+    Model *m = quantized(h);
+    if (!m) return IM_ERR_INVALID;
     if (m->world <= 1) return IM_OK;
 #if IM_HAVE_NCCL_H
     if (!nccl()) return fail(IM_ERR_NCCL, "libnccl.so.2 could not be loaded");
@@ -1183,7 +963,7 @@ IM_EXPORT int im_cuda_model_create(im_device *dev, const im_model_config *cfg, i
     if (c.prefill_chunk_size == 0) c.prefill_chunk_size = kPrefillChunk;
     if (c.prefill_chunk_size > c.max_seq_len) c.prefill_chunk_size = c.max_seq_len;  // no prompt is longer than the cache
     IM_CUDA_CHECK(cudaSetDevice(dev->ordinal));
-    im_model *m = new im_model();
+    Model *m = new Model();
     m->dev = dev;
     m->cfg = c;
     m->world = c.tp_world;
@@ -1196,48 +976,23 @@ IM_EXPORT int im_cuda_model_create(im_device *dev, const im_model_config *cfg, i
     m->kv_dim = m->nkv_l * c.head_dim;
     m->qkv_dim = m->q_dim + 2 * m->kv_dim;
     m->layers.resize(c.num_layers);
-    cudaError_t e = cudaStreamCreateWithFlags(&m->stream, cudaStreamNonBlocking);
-    if (e != cudaSuccess) {
+    m->logit_parts = m->world;
+    const int orc = session_open(m);
+    if (orc != IM_OK) {
         delete m;
-        return fail(IM_ERR_CUDA, "stream creation failed: %s", cudaGetErrorString(e));
+        return orc;
     }
     *out = m;
     return IM_OK;
     IM_GUARD_END
 }
 
-IM_EXPORT void im_cuda_model_free(im_model *m) {
-    if (!m) return;
-    cudaSetDevice(m->dev->ordinal);
-    if (m->stream) cudaStreamSynchronize(m->stream);
-    for (auto &g : m->graphs) cudaGraphExecDestroy(g.second);
-#if IM_HAVE_NCCL_H
-    for (int p = 0; p < kXarMaxWorld; p++)
-        if (m->xar.peer[p] && p != m->rank) cudaIpcCloseMemHandle(m->xar.peer[p]);
-    if (m->xar.base) cudaFree(m->xar.base);
-    if (m->comm && nccl() && nccl()->CommDestroy) nccl()->CommDestroy(m->comm);
-#endif
-    for (auto &L : m->layers) {
-        im_cuda_affine_weight_free(static_cast<im_affine_weight *>(L.qkv));
-        im_cuda_affine_weight_free(static_cast<im_affine_weight *>(L.o));
-        im_cuda_affine_weight_free(static_cast<im_affine_weight *>(L.gate));
-        im_cuda_affine_weight_free(static_cast<im_affine_weight *>(L.up));
-        im_cuda_affine_weight_free(static_cast<im_affine_weight *>(L.down));
-    }
-    if (m->tq) im_cuda_tq_free(m->tq);
-    for (auto &a : m->allocs) dev_free(m->dev, a.first, a.second);
-    if (m->tokens_pin) cudaFreeHost(m->tokens_pin);
-    if (m->logits_pin) cudaFreeHost(m->logits_pin);
-    if (m->logits_seq_pin) cudaFreeHost(m->logits_seq_pin);
-    if (m->slot_pin) cudaFreeHost(m->slot_pin);
-    if (m->err_pin) cudaFreeHost(m->err_pin);
-    if (m->stream) cudaStreamDestroy(m->stream);
-    delete m;
-}
 
-IM_EXPORT int im_cuda_model_load_dense(im_model *m, const char *name, const void *data_f16_host, size_t n) {
+IM_EXPORT int im_cuda_model_load_dense(im_model *h, const char *name, const void *data_f16_host, size_t n) {
     IM_GUARD_BEGIN
-    IM_REQUIRE(m && name && data_f16_host, "bad argument");
+    IM_REQUIRE(h && name && data_f16_host, "bad argument");
+    Model *m = quantized(h);
+    if (!m) return IM_ERR_INVALID;
     if (m->finalized) return fail(IM_ERR_STATE, "model already finalized");
     IM_CUDA_CHECK(cudaSetDevice(m->dev->ordinal));
     const im_model_config &c = m->cfg;
@@ -1270,11 +1025,13 @@ IM_EXPORT int im_cuda_model_load_dense(im_model *m, const char *name, const void
     IM_GUARD_END
 }
 
-IM_EXPORT int im_cuda_model_load_affine(im_model *m, const char *name, const void *qdata_host, const void *scales_host,
+IM_EXPORT int im_cuda_model_load_affine(im_model *h, const char *name, const void *qdata_host, const void *scales_host,
                                         const void *zeros_host, int param_dtype, const void *awq_f16_host, int N, int K,
                                         int group_size, int bit_width) {
     IM_GUARD_BEGIN
-    IM_REQUIRE(m && name && qdata_host && scales_host && zeros_host, "bad argument");
+    IM_REQUIRE(h && name && qdata_host && scales_host && zeros_host, "bad argument");
+    Model *m = quantized(h);
+    if (!m) return IM_ERR_INVALID;
     if (m->finalized) return fail(IM_ERR_STATE, "model already finalized");
     IM_REQUIRE(bit_width == 4 || bit_width == 8, "bit_width must be 4 or 8");
     IM_REQUIRE(group_size > 0, "group_size must be positive");
@@ -1329,9 +1086,11 @@ IM_EXPORT int im_cuda_model_load_affine(im_model *m, const char *name, const voi
     IM_GUARD_END
 }
 
-IM_EXPORT int im_cuda_model_set_tq_constants(im_model *m, const float *signs_host, const float *qjl_host) {
+IM_EXPORT int im_cuda_model_set_tq_constants(im_model *h, const float *signs_host, const float *qjl_host) {
     IM_GUARD_BEGIN
-    IM_REQUIRE(m && signs_host && qjl_host, "bad argument");
+    IM_REQUIRE(h && signs_host && qjl_host, "bad argument");
+    Model *m = quantized(h);
+    if (!m) return IM_ERR_INVALID;
     if (m->finalized) return fail(IM_ERR_STATE, "model already finalized");
     const size_t hd = m->cfg.head_dim;
     m->signs_host.assign(signs_host, signs_host + hd);
@@ -1340,11 +1099,8 @@ IM_EXPORT int im_cuda_model_set_tq_constants(im_model *m, const float *signs_hos
     IM_GUARD_END
 }
 
-IM_EXPORT int im_cuda_model_finalize(im_model *m) {
-    IM_GUARD_BEGIN
-    IM_REQUIRE(m, "bad argument");
-    if (m->finalized) return IM_OK;
-    IM_CUDA_CHECK(cudaSetDevice(m->dev->ordinal));
+int Model::finalize() {
+    Model *const m = this;
     const im_model_config &c = m->cfg;
     const int H = c.hidden_size, hd = c.head_dim;
     if (!m->embed) return fail(IM_ERR_STATE, "missing tensor model.embed_tokens.weight");
@@ -1429,30 +1185,8 @@ IM_EXPORT int im_cuda_model_finalize(im_model *m) {
             if (!w || (w->bits != 4 && w->bits != 8) || w->group_size != 128 || w->K % 128 != 0 || w->N % 8 != 0) m->gemm_ok = false;
     IM_TRY(m->alloc((void **)&m->logits, (size_t)c.max_batch * m->vocab_l * 2));
     if (m->world > 1) IM_TRY(m->alloc((void **)&m->logits_all, (size_t)c.max_batch * c.vocab_size * 2));
-    IM_TRY(m->alloc((void **)&m->tokens_dev, MT * 4));
-    IM_TRY(m->alloc((void **)&m->tok_hist, (size_t)c.max_seq_len * c.max_batch * 4));
-    IM_TRY(m->alloc((void **)&m->pos_dev, 64 * 4));
-    IM_TRY(m->alloc((void **)&m->slot_ident, 64 * 4));
-    IM_TRY(m->alloc((void **)&m->slot_map, 64 * 4));
-    {
-        int ident[64];
-        for (int i = 0; i < 64; i++) ident[i] = i;
-        IM_CUDA_CHECK(cudaMemcpy(m->slot_ident, ident, sizeof(ident), cudaMemcpyHostToDevice));
-        IM_CUDA_CHECK(cudaMemcpy(m->slot_map, ident, sizeof(ident), cudaMemcpyHostToDevice));
-    }
-    IM_CUDA_CHECK(cudaMallocHost((void **)&m->slot_pin, 64 * sizeof(int)));
-    m->slot_pos.assign((size_t)c.max_batch, 0);
-    m->slot_used.assign((size_t)c.max_batch, 0);
-    IM_TRY(m->alloc((void **)&m->step_dev, 4));
-    IM_CUDA_CHECK(cudaMemset(m->pos_dev, 0, 64 * 4));
-    IM_CUDA_CHECK(cudaMemset(m->step_dev, 0, 4));
-    IM_TRY(m->alloc((void **)&m->argmax_cand, (size_t)c.max_batch * kArgmaxCtas * sizeof(float2)));
-    IM_TRY(m->alloc((void **)&m->argmax_counters, (size_t)c.max_batch * sizeof(unsigned)));
-    IM_CUDA_CHECK(cudaMemset(m->argmax_counters, 0, (size_t)c.max_batch * sizeof(unsigned)));
-    IM_CUDA_CHECK(cudaMallocHost((void **)&m->tokens_pin, MT * 4));
-    IM_CUDA_CHECK(cudaMallocHost((void **)&m->logits_pin, (size_t)c.max_batch * c.vocab_size * 2));
-    IM_CUDA_CHECK(cudaMallocHost((void **)&m->err_pin, sizeof(int)));
-    *m->err_pin = 0;
+    m->logits_dev = m->world > 1 ? m->logits_all : m->logits;
+    IM_TRY(session_alloc(m));
     // attention scratch for the largest launch: decode at max_batch, or a prefill chunk
     size_t need = 0;
     for (int b = 1; b <= c.max_batch; b++) {
@@ -1465,8 +1199,8 @@ IM_EXPORT int im_cuda_model_finalize(im_model *m) {
     }
     if (c.tq_bits == 16) {
         size_t n16 = 0;
-        for (int b = 1; b <= c.max_batch; b++) n16 = std::max(n16, kv16_scratch_bytes(b, m->nh_l, kv16_auto_splits(m->dev, b, m->nkv_l, c.max_seq_len)));
-        for (int t = 1; t <= m->MT; t++) n16 = std::max(n16, kv16_scratch_bytes(t, m->nh_l, kv16_auto_splits(m->dev, t, m->nkv_l, c.max_seq_len)));
+        for (int b = 1; b <= c.max_batch; b++) n16 = std::max(n16, im::kv16_scratch_bytes(b, m->nh_l, kv16_auto_splits(m->dev, b, m->nkv_l, c.max_seq_len)));
+        for (int t = 1; t <= m->MT; t++) n16 = std::max(n16, im::kv16_scratch_bytes(t, m->nh_l, kv16_auto_splits(m->dev, t, m->nkv_l, c.max_seq_len)));
         IM_TRY(m->alloc((void **)&m->kv16_scratch, n16));
         m->kv16_scratch_bytes = n16;
     }
@@ -1477,61 +1211,18 @@ IM_EXPORT int im_cuda_model_finalize(im_model *m) {
     m->bytes += need + reinterpret_cast<Tq *>(m->tq)->const_bytes;
     IM_CUDA_CHECK(cudaDeviceSynchronize());
     IM_TRY(mega_prepare(m));
-    m->finalized = true;
     return IM_OK;
-    IM_GUARD_END
 }
 
-IM_EXPORT int im_cuda_model_reset(im_model *m) {
-    IM_GUARD_BEGIN
-    IM_REQUIRE(m, "bad argument");
-    if (!m->finalized) return fail(IM_ERR_STATE, "model not loaded");
-    IM_CUDA_CHECK(cudaSetDevice(m->dev->ordinal));
-    for (char &u : m->slot_used) u = 0;
-    return set_positions(m, 0);
-    IM_GUARD_END
-}
-
-IM_EXPORT int im_cuda_model_truncate(im_model *m, int pos) {
-    IM_GUARD_BEGIN
-    IM_REQUIRE(m, "bad argument");
-    if (!m->finalized) return fail(IM_ERR_STATE, "model not loaded");
-    if (pos < 0 || pos > m->slot_pos[0]) return fail(IM_ERR_BOUNDS, "truncate_to(%d) is outside the current sequence of %d tokens", pos, m->slot_pos[0]);
-    IM_CUDA_CHECK(cudaSetDevice(m->dev->ordinal));
-    return set_positions(m, pos);
-    IM_GUARD_END
-}
-
-// The final RMSNorm output the lm_head consumed in the last step (norm_out of
-// crates/ironmill-inference/src/metal/pipeline.rs:176-226, decode_step_with_hidden / last_hidden_state), fp16 widened
-// to f32: `rows` rows of hidden_size, one per sequence of that step in its order (row 0 for the single-sequence calls;
-// after prefill_all_logits: one row per token of the last chunk).
-IM_EXPORT int im_cuda_model_last_hidden_state(im_model *m, int rows, float *out_host) {
-    IM_GUARD_BEGIN
-    IM_REQUIRE(m && out_host, "bad argument");
-    if (!m->finalized) return fail(IM_ERR_STATE, "model not loaded");
-    const int cap = m->MT;
-    if (rows < 1 || rows > cap) return fail(IM_ERR_BOUNDS, "rows must be in 1..%d, got %d", cap, rows);
-    IM_CUDA_CHECK(cudaSetDevice(m->dev->ordinal));
-    const size_t n = (size_t)rows * m->cfg.hidden_size;
-    std::vector<__half> tmp(n);
-    IM_CUDA_CHECK(cudaMemcpyAsync(tmp.data(), m->norm_out, n * sizeof(__half), cudaMemcpyDeviceToHost, m->stream));
-    IM_CUDA_CHECK(cudaStreamSynchronize(m->stream));
-    for (size_t i = 0; i < n; i++) out_host[i] = __half2float(tmp[i]);
-    return IM_OK;
-    IM_GUARD_END
-}
-
-IM_EXPORT int im_cuda_model_seq_pos(const im_model *m) { return m && !m->slot_pos.empty() ? m->slot_pos[0] : 0; }
-IM_EXPORT int im_cuda_model_max_seq_len(const im_model *m) { return m ? m->cfg.max_seq_len : 0; }
-IM_EXPORT size_t im_cuda_model_memory_bytes(const im_model *m) { return m ? m->bytes : 0; }
 // Timing of the whole-token decode kernel alone: `reps` launches back to back on the model's stream between two
 // events (the sequence position is not advanced: every launch rewrites the same cache row), and the time CTA 0
 // spent in each of the seven phases of a layer, averaged over the layers of the last launch, from the
 // nanosecond-timer stamps it leaves at every grid barrier.  IM_ERR_STATE when the model does not use that kernel.
-IM_EXPORT int im_cuda_model_token_kernel_profile(im_model *m, int reps, float *ms_per_launch, float *phase_us_7) {
+IM_EXPORT int im_cuda_model_token_kernel_profile(im_model *h, int reps, float *ms_per_launch, float *phase_us_7) {
     IM_GUARD_BEGIN
-    IM_REQUIRE(m && reps >= 1 && ms_per_launch, "bad argument");
+    IM_REQUIRE(h && reps >= 1 && ms_per_launch, "bad argument");
+    Model *m = quantized(h);
+    if (!m) return IM_ERR_INVALID;
     if (!m->finalized) return fail(IM_ERR_STATE, "model not loaded");
     if (!m->mega_ready) return fail(IM_ERR_STATE, "this model does not run the whole-token decode kernel");
     if (m->slot_pos[0] + 1 > m->cfg.max_seq_len) return fail(IM_ERR_BOUNDS, "no room for one more position");
@@ -1556,7 +1247,7 @@ IM_EXPORT int im_cuda_model_token_kernel_profile(im_model *m, int reps, float *m
     cudaEventDestroy(e1);
     IM_TRY(rc);
     if (e != cudaSuccess) return fail(IM_ERR_CUDA, "whole-token kernel failed: %s", cudaGetErrorString(e));
-    IM_TRY(step_error_check(m));
+    IM_TRY(session_error_check(m));
     *ms_per_launch = ms / (float)reps;
     if (phase_us_7) {
         const int L = c.num_layers, n = 7 * L + 2;
@@ -1578,9 +1269,11 @@ IM_EXPORT int im_cuda_model_token_kernel_profile(im_model *m, int reps, float *m
 
 // Test hook of the error path: see the header.  The captured decode graphs hold the kernel's parameters by value, so
 // they are dropped and the next step captures again.
-IM_EXPORT int im_cuda_model_test_missing_ranks(im_model *m, int missing_ranks) {
+IM_EXPORT int im_cuda_model_test_missing_ranks(im_model *h, int missing_ranks) {
     IM_GUARD_BEGIN
-    IM_REQUIRE(m && (missing_ranks == 0 || missing_ranks == 1), "bad argument");
+    IM_REQUIRE(h && (missing_ranks == 0 || missing_ranks == 1), "bad argument");
+    Model *m = quantized(h);
+    if (!m) return IM_ERR_INVALID;
     if (!m->finalized) return fail(IM_ERR_STATE, "model not loaded");
     if (!m->mega_ready || !m->mega_capacity2 || m->world != 1)
         return fail(IM_ERR_STATE, "only for a single-GPU model loaded with decode_schedule = 2");
@@ -1596,222 +1289,8 @@ IM_EXPORT int im_cuda_model_test_missing_ranks(im_model *m, int missing_ranks) {
 
 // 1 when the row-split projections of a tensor-parallel model are summed by the one-shot peer-memory all-reduce,
 // 0 when NCCL does it (single GPU: 0).
-IM_EXPORT int im_cuda_model_tp_peer_allreduce(const im_model *m) { return m && m->xar.ok ? 1 : 0; }
-IM_EXPORT int im_cuda_model_token_kernel(const im_model *m) { return m && m->mega_ready ? 1 : 0; }
-IM_EXPORT int im_cuda_model_step_launches(const im_model *m) { return m ? m->launches_per_step : 0; }
-
-IM_EXPORT size_t im_cuda_model_step_bytes(const im_model *m, int ctx, int batch) {
-    if (!m || !m->finalized) return 0;
-    const im_model_config &c = m->cfg;
-    size_t b = 0;
-    for (const Layer &L : m->layers) {
-        for (const AffineWeight *w : {L.qkv, L.o, L.gate, L.up, L.down}) {
-            b += (size_t)w->N * w->K * w->bits / 8 + (size_t)w->N * w->G * 4 + (w->awq ? (size_t)w->K * 2 : 0);
-        }
-        b += 2 * (size_t)c.hidden_size * 2;
-        b += (size_t)batch * m->nkv_l * ctx * (2 * c.head_dim * c.tq_bits / 8 + (c.tq_bits == 16 ? 0 : 12));
-    }
-    b += (size_t)m->vocab_l * c.hidden_size * 2 + (size_t)c.hidden_size * 2;
-    return b;
-}
-
-IM_EXPORT int im_cuda_model_prefill(im_model *m, const uint32_t *tokens_host, int n, float *logits_out_host) {
-    IM_GUARD_BEGIN
-    IM_REQUIRE(m && tokens_host && logits_out_host, "bad argument");
-    if (!m->finalized) return fail(IM_ERR_STATE, "model not loaded");
-    IM_REQUIRE(n > 0, "prefill needs at least one token");
-    IM_CUDA_CHECK(cudaSetDevice(m->dev->ordinal));
-    return prefill_slot(m, 0, tokens_host, n, logits_out_host, nullptr);
-    IM_GUARD_END
-}
-
-IM_EXPORT int im_cuda_model_prefill_all_logits(im_model *m, const uint32_t *tokens_host, int n, float *logits_out_host) {
-    IM_GUARD_BEGIN
-    IM_REQUIRE(m && tokens_host && logits_out_host, "bad argument");
-    if (!m->finalized) return fail(IM_ERR_STATE, "model not loaded");
-    IM_REQUIRE(n > 0, "prefill needs at least one token");
-    IM_CUDA_CHECK(cudaSetDevice(m->dev->ordinal));
-    return prefill_slot(m, 0, tokens_host, n, nullptr, logits_out_host);
-    IM_GUARD_END
-}
-
-// ---- continuous batching: BatchInferenceEngine (crates/ironmill-inference/src/engine.rs:121-131) -------------------
-IM_EXPORT int im_cuda_model_seq_add(im_model *m, const uint32_t *tokens_host, int n, int *seq_id_out, float *logits_out_host) {
-    IM_GUARD_BEGIN
-    IM_REQUIRE(m && tokens_host && seq_id_out, "bad argument");
-    if (!m->finalized) return fail(IM_ERR_STATE, "model not loaded");
-    IM_REQUIRE(n > 0, "a sequence needs at least one prompt token");
-    int slot = -1;
-    for (int s = 0; s < m->cfg.max_batch && slot < 0; s++)
-        if (!m->slot_used[s]) slot = s;
-    if (slot < 0) return fail(IM_ERR_BOUNDS, "all %d sequence slots are in use (max_batch)", m->cfg.max_batch);
-    IM_CUDA_CHECK(cudaSetDevice(m->dev->ordinal));
-    set_one_pos_kernel<<<1, 1, 0, m->stream>>>(m->pos_dev, slot, 0);
-    IM_CUDA_CHECK(cudaGetLastError());
-    m->slot_pos[slot] = 0;
-    int rc = prefill_slot(m, slot, tokens_host, n, logits_out_host, nullptr);
-    if (rc != IM_OK) return rc;
-    m->slot_used[slot] = 1;
-    *seq_id_out = slot;
-    return IM_OK;
-    IM_GUARD_END
-}
-
-IM_EXPORT int im_cuda_model_seq_remove(im_model *m, int seq_id) {
-    IM_GUARD_BEGIN
-    IM_REQUIRE(m, "bad argument");
-    if (!m->finalized) return fail(IM_ERR_STATE, "model not loaded");
-    if (seq_id < 0 || seq_id >= m->cfg.max_batch || !m->slot_used[seq_id]) return fail(IM_ERR_INVALID, "no sequence %d", seq_id);
-    m->slot_used[seq_id] = 0;   // the slot's cache rows are simply overwritten by the next tenant
-    m->slot_pos[seq_id] = 0;
-    return IM_OK;
-    IM_GUARD_END
-}
-
-IM_EXPORT int im_cuda_model_seq_position(const im_model *m, int seq_id) {
-    if (!m || seq_id < 0 || seq_id >= (int)m->slot_pos.size() || !m->slot_used[seq_id]) return -1;
-    return m->slot_pos[seq_id];
-}
-
-// One decode step for the listed sequences (any subset of the live ones, each at its own position): tokens_host[i] is
-// appended to sequence seq_ids[i]; logits_out_host f32 [n, vocab] in the same order.
-IM_EXPORT int im_cuda_model_batch_decode_step(im_model *m, const int *seq_ids, const uint32_t *tokens_host, int n, float *logits_out_host) {
-    IM_GUARD_BEGIN
-    IM_REQUIRE(m && seq_ids && tokens_host && logits_out_host, "bad argument");
-    if (!m->finalized) return fail(IM_ERR_STATE, "model not loaded");
-    IM_REQUIRE(n >= 1 && n <= m->cfg.max_batch, "batch %d outside 1..max_batch (%d)", n, m->cfg.max_batch);
-    for (int i = 0; i < n; i++) {
-        const int s = seq_ids[i];
-        if (s < 0 || s >= m->cfg.max_batch || !m->slot_used[s]) return fail(IM_ERR_INVALID, "no sequence %d", s);
-        for (int j = 0; j < i; j++)
-            if (seq_ids[j] == s) return fail(IM_ERR_INVALID, "sequence %d listed twice", s);
-        if (m->slot_pos[s] + 1 > m->cfg.max_seq_len)
-            return fail(IM_ERR_BOUNDS, "sequence %d: position %d + 1 exceeds max_seq_len %d", s, m->slot_pos[s], m->cfg.max_seq_len);
-    }
-    IM_CUDA_CHECK(cudaSetDevice(m->dev->ordinal));
-    cudaStream_t st = m->stream;
-    memcpy(m->slot_pin, seq_ids, (size_t)n * sizeof(int));
-    IM_CUDA_CHECK(cudaMemcpyAsync(m->slot_map, m->slot_pin, (size_t)n * sizeof(int), cudaMemcpyHostToDevice, st));
-    cudaGraphExec_t g = nullptr;
-    IM_TRY(get_graph(m, n, &g, true));
-    memcpy(m->tokens_pin, tokens_host, (size_t)n * 4);
-    IM_CUDA_CHECK(cudaMemcpyAsync(m->tokens_dev, m->tokens_pin, (size_t)n * 4, cudaMemcpyHostToDevice, st));
-    IM_CUDA_CHECK(cudaGraphLaunch(g, st));
-    const __half *lg = m->world > 1 ? m->logits_all : m->logits;
-    IM_CUDA_CHECK(cudaMemcpyAsync(m->logits_pin, lg, (size_t)n * m->cfg.vocab_size * 2, cudaMemcpyDeviceToHost, st));
-    IM_CUDA_CHECK(cudaMemcpyAsync(m->err_pin, m->dev->err_flag, sizeof(int), cudaMemcpyDeviceToHost, st));
-    IM_CUDA_CHECK(cudaStreamSynchronize(st));
-    IM_TRY(step_error_check(m));
-    for (int i = 0; i < n; i++) m->slot_pos[seq_ids[i]] += 1;
-    logits_to_host(m, m->logits_pin, n, logits_out_host);
-    return IM_OK;
-    IM_GUARD_END
-}
-
-IM_EXPORT int im_cuda_model_decode_step(im_model *m, const uint32_t *tokens_host, int batch, float *logits_out_host) {
-    IM_GUARD_BEGIN
-    IM_REQUIRE(m && tokens_host && logits_out_host, "bad argument");
-    if (!m->finalized) return fail(IM_ERR_STATE, "model not loaded");
-    IM_REQUIRE(batch >= 1 && batch <= m->cfg.max_batch, "batch %d outside 1..max_batch (%d)", batch, m->cfg.max_batch);
-    int far = 0;
-    for (int b = 0; b < batch; b++) far = m->slot_pos[b] > far ? m->slot_pos[b] : far;
-    if (far + 1 > m->cfg.max_seq_len)
-        return fail(IM_ERR_BOUNDS, "sequence position %d + 1 exceeds max_seq_len %d", far, m->cfg.max_seq_len);
-    IM_CUDA_CHECK(cudaSetDevice(m->dev->ordinal));
-    cudaStream_t st = m->stream;
-    cudaGraphExec_t g = nullptr;
-    IM_TRY(get_graph(m, batch, &g));
-    memcpy(m->tokens_pin, tokens_host, (size_t)batch * 4);
-    IM_CUDA_CHECK(cudaMemcpyAsync(m->tokens_dev, m->tokens_pin, (size_t)batch * 4, cudaMemcpyHostToDevice, st));
-    IM_CUDA_CHECK(cudaGraphLaunch(g, st));
-    const __half *lg = m->world > 1 ? m->logits_all : m->logits;
-    IM_CUDA_CHECK(cudaMemcpyAsync(m->logits_pin, lg, (size_t)batch * m->cfg.vocab_size * 2, cudaMemcpyDeviceToHost, st));
-    IM_CUDA_CHECK(cudaMemcpyAsync(m->err_pin, m->dev->err_flag, sizeof(int), cudaMemcpyDeviceToHost, st));
-    IM_CUDA_CHECK(cudaStreamSynchronize(st));
-    IM_TRY(step_error_check(m));
-    for (int b = 0; b < batch; b++) m->slot_pos[b] += 1;
-    logits_to_host(m, m->logits_pin, batch, logits_out_host);
-    return IM_OK;
-    IM_GUARD_END
-}
-
-IM_EXPORT int im_cuda_model_decode_greedy(im_model *m, const uint32_t *first_tokens_host, int batch, int n_steps,
-                                          uint32_t *tokens_out_host, float *elapsed_ms_out) {
-    IM_GUARD_BEGIN
-    IM_REQUIRE(m && first_tokens_host, "bad argument");
-    if (!m->finalized) return fail(IM_ERR_STATE, "model not loaded");
-    IM_REQUIRE(batch >= 1 && batch <= m->cfg.max_batch, "batch %d outside 1..max_batch (%d)", batch, m->cfg.max_batch);
-    IM_REQUIRE(n_steps >= 0, "n_steps must be >= 0");
-    int far = 0;
-    for (int b = 0; b < batch; b++) far = m->slot_pos[b] > far ? m->slot_pos[b] : far;
-    if (far + n_steps > m->cfg.max_seq_len)
-        return fail(IM_ERR_BOUNDS, "sequence position %d + %d steps exceeds max_seq_len %d", far, n_steps, m->cfg.max_seq_len);
-    IM_CUDA_CHECK(cudaSetDevice(m->dev->ordinal));
-    cudaStream_t st = m->stream;
-    cudaGraphExec_t g = nullptr;
-    IM_TRY(get_graph(m, batch, &g));
-    memcpy(m->tokens_pin, first_tokens_host, (size_t)batch * 4);
-    IM_CUDA_CHECK(cudaMemcpyAsync(m->tokens_dev, m->tokens_pin, (size_t)batch * 4, cudaMemcpyHostToDevice, st));
-    IM_CUDA_CHECK(cudaMemsetAsync(m->step_dev, 0, 4, st));
-    cudaEvent_t e0, e1;
-    IM_CUDA_CHECK(cudaEventCreate(&e0));
-    IM_CUDA_CHECK(cudaEventCreate(&e1));
-    cudaEventRecord(e0, st);
-    for (int i = 0; i < n_steps; i++) {
-        cudaError_t e = cudaGraphLaunch(g, st);
-        if (e != cudaSuccess) {
-            cudaEventDestroy(e0);
-            cudaEventDestroy(e1);
-            return fail(IM_ERR_CUDA, "graph launch failed: %s", cudaGetErrorString(e));
-        }
-    }
-    cudaEventRecord(e1, st);
-    cudaMemcpyAsync(m->err_pin, m->dev->err_flag, sizeof(int), cudaMemcpyDeviceToHost, st);
-    cudaError_t e = cudaStreamSynchronize(st);
-    float ms = 0.0f;
-    cudaEventElapsedTime(&ms, e0, e1);
-    cudaEventDestroy(e0);
-    cudaEventDestroy(e1);
-    if (e != cudaSuccess) return fail(IM_ERR_CUDA, "decode loop failed: %s", cudaGetErrorString(e));
-    IM_TRY(step_error_check(m));
-    for (int b = 0; b < batch; b++) m->slot_pos[b] += n_steps;
-    if (elapsed_ms_out) *elapsed_ms_out = ms;
-    if (tokens_out_host && n_steps > 0)
-        IM_CUDA_CHECK(cudaMemcpy2D(tokens_out_host, (size_t)batch * 4, m->tok_hist, (size_t)m->cfg.max_batch * 4, (size_t)batch * 4, n_steps,
-                                   cudaMemcpyDeviceToHost));
-    return IM_OK;
-    IM_GUARD_END
-}
-
-IM_EXPORT int im_cuda_model_profile_step(im_model *m, int batch, float *ms_by_category, int n_categories) {
-    IM_GUARD_BEGIN
-    IM_REQUIRE(m && ms_by_category && n_categories >= kCatCount, "bad argument (need %d categories)", (int)kCatCount);
-    if (!m->finalized) return fail(IM_ERR_STATE, "model not loaded");
-    IM_REQUIRE(batch >= 1 && batch <= m->cfg.max_batch, "batch %d outside 1..max_batch (%d)", batch, m->cfg.max_batch);
-    for (int b = 0; b < batch; b++)
-        if (m->slot_pos[b] + 1 > m->cfg.max_seq_len) return fail(IM_ERR_BOUNDS, "no room for one more position");
-    IM_CUDA_CHECK(cudaSetDevice(m->dev->ordinal));
-    cudaStream_t st = m->stream;
-    const int splits = decode_splits(m, batch);
-    IM_TRY(forward(m, batch, 1, splits, st, nullptr));  // warm
-    Prof prof;
-    prof.st = st;
-    prof.mark(-1);
-    int rc = forward(m, batch, 1, splits, st, nullptr, &prof);
-    cudaError_t e = cudaStreamSynchronize(st);
-    for (int i = 0; i < n_categories; i++) ms_by_category[i] = 0.0f;
-    if (rc == IM_OK && e == cudaSuccess)
-        for (size_t i = 1; i < prof.ev.size(); i++) {
-            float ms = 0.0f;
-            cudaEventElapsedTime(&ms, prof.ev[i - 1], prof.ev[i]);
-            ms_by_category[prof.cat[i]] += ms;
-        }
-    for (cudaEvent_t ev : prof.ev) cudaEventDestroy(ev);
-    if (rc != IM_OK) return rc;
-    if (e != cudaSuccess) return fail(IM_ERR_CUDA, "profile step failed: %s", cudaGetErrorString(e));
-    return IM_OK;
-    IM_GUARD_END
-}
+IM_EXPORT int im_cuda_model_tp_peer_allreduce(const im_model *h) { const Model *m = quantized(h); return m && m->xar.ok ? 1 : 0; }
+IM_EXPORT int im_cuda_model_token_kernel(const im_model *h) { const Model *m = quantized(h); return m && m->mega_ready ? 1 : 0; }
 
 // Host-only helpers of the tensor-parallel loader, exported so that the shard arithmetic can be checked on a
 // machine without a GPU.  `suffix` is the part of the tensor name after "model.layers.<i>.".

@@ -13,8 +13,9 @@ from dataclasses import dataclass
 
 import numpy as np
 
-from ._lib import CudaSysError, IM_DTYPE_F16, IM_DTYPE_F32, check, lib, vp
-from .bundle import ModelConfig, WeightTensor
+from ._lib import CudaSysError, check, lib, vp
+from .architectures import _CModelConfig, family_of  # noqa: F401  (_CModelConfig: layout of im_model_config)
+from .bundle import GpuBundleError, WeightTensor
 
 
 class InferenceError(RuntimeError):
@@ -32,6 +33,8 @@ def _wrap(fn):
         except CudaSysError as e:  # backend error converts like From<MetalError> (metal/error.rs:47-51)
             kind = {-3: "Allocation", -7: "NotLoaded", -4: "Decode"}.get(e.code, "Runtime")
             raise InferenceError(kind, e.message) from e
+        except GpuBundleError as e:
+            raise InferenceError("Runtime", str(e)) from e
     return inner
 
 
@@ -52,6 +55,7 @@ class CudaConfig:
     decode_schedule: str = "auto"
     tp_collective: str = "auto"   # "auto" (peer-memory exchange when the ranks can map each other) or "nccl"
     wait_limit_ms: int = 0        # patience of device-side bounded waits (0 = default)
+    dtype: str = "bfloat16"       # list-of-layers models: "bfloat16" or "float32" (everything in true 32-bit)
 
     def with_max_seq_len(self, n: int) -> "CudaConfig":
         self.max_seq_len = n
@@ -71,16 +75,8 @@ class CudaConfig:
             raise InferenceError("Runtime", "max_seq_len must be > 0")
         if self.n_bits not in (4, 8):
             raise InferenceError("Runtime", f"n_bits must be 4 or 8, got {self.n_bits}")
-
-
-class _CModelConfig(C.Structure):
-    _fields_ = [("num_layers", C.c_int), ("hidden_size", C.c_int), ("intermediate_size", C.c_int), ("num_heads", C.c_int),
-                ("num_kv_heads", C.c_int), ("head_dim", C.c_int), ("vocab_size", C.c_int), ("max_seq_len", C.c_int),
-                ("max_batch", C.c_int), ("rms_eps", C.c_float), ("attn_scale", C.c_float), ("embed_scale", C.c_float),
-                ("rope_theta", C.c_double), ("rotary_dim", C.c_int), ("qk_norm", C.c_int), ("tie_word_embeddings", C.c_int),
-                ("tq_bits", C.c_int), ("rotation_seed", C.c_uint64), ("tp_world", C.c_int), ("tp_rank", C.c_int),
-                ("prefill_chunk_size", C.c_int), ("decode_schedule", C.c_int), ("tp_collective", C.c_int),
-                ("wait_limit_ms", C.c_int)]
+        if self.dtype not in ("bfloat16", "float32"):
+            raise InferenceError("Runtime", f"dtype must be bfloat16 or float32, got {self.dtype}")
 
 
 @dataclass
@@ -109,7 +105,7 @@ class CudaInference:
         self.config.validate()
         self._dev = C.c_void_p()
         self._model = C.c_void_p()
-        self._mc: ModelConfig | None = None
+        self._mc = None
         try:
             check(lib().im_cuda_device_open(C.c_int(self.config.device), C.byref(self._dev)))
         except CudaSysError as e:
@@ -126,55 +122,22 @@ class CudaInference:
         if self._model:
             lib().im_cuda_model_free(self._model)
             self._model = C.c_void_p()
-        mc: ModelConfig = provider.config()
-        self._mc = mc
-        cc = _CModelConfig(mc.num_hidden_layers, mc.hidden_size, mc.intermediate_size, mc.num_attention_heads,
-                           mc.num_key_value_heads, mc.head_dim, mc.vocab_size, self.config.max_seq_len, self.config.max_batch,
-                           mc.rms_norm_eps, mc.attn_scale, float(mc.extra.get("embed_scale", 0.0) or 0.0), mc.rope_theta,
-                           int(mc.extra.get("rotary_dim", 0) or 0), int(mc.has_qk_norm), int(mc.tie_word_embeddings),
-                           self.config.n_bits if self.config.enable_turboquant else 16, self.config.rotation_seed, self.config.tp_world,
-                           self.config.tp_rank,
-                           int(self.config.prefill_chunk_size or 0),
-                           {"auto": 0, "per_kernel": 1, "tagged": 2}[self.config.decode_schedule],
-                           {"auto": 0, "nccl": 1}[self.config.tp_collective], int(self.config.wait_limit_ms))
-        check(lib().im_cuda_model_create(self._dev, C.byref(cc), C.byref(self._model)))
+        mc = provider.config()
+        family = family_of(mc)
+        self._mc, self._family = mc, family
+        self._model = family.create(self, mc)
         if tq_signs is not None:
             s = np.ascontiguousarray(tq_signs, dtype=np.float32)
             q = np.ascontiguousarray(tq_qjl, dtype=np.float32)
             check(lib().im_cuda_model_set_tq_constants(self._model, vp(s), vp(q)))
-        names = ["model.embed_tokens.weight", "model.norm.weight"]
-        if provider.has_tensor("lm_head.weight"):
-            names.append("lm_head.weight")
-        for i in range(mc.num_hidden_layers):
-            p = f"model.layers.{i}"
-            names += [f"{p}.input_layernorm.weight", f"{p}.post_attention_layernorm.weight"]
-            if mc.has_qk_norm:
-                names += [f"{p}.self_attn.q_norm.weight", f"{p}.self_attn.k_norm.weight"]
-            names += [f"{p}.self_attn.{x}_proj.weight" for x in "qkvo"] + [f"{p}.mlp.{x}_proj.weight" for x in ("gate", "up", "down")]
-        for name in names:
+        for name in family.tensor_names(mc, provider):
             if not provider.has_tensor(name):
                 raise InferenceError("Runtime", f"weight provider has no tensor '{name}'")
             self._load_tensor(name, provider.tensor(name))
         check(lib().im_cuda_model_finalize(self._model))
 
     def _load_tensor(self, name: str, t: WeightTensor) -> None:
-        if not t.quantized:
-            data = np.ascontiguousarray(t.data)
-            if data.dtype != np.float16:
-                data = data.astype(np.float16)   # dense tensors live in fp16 on the GPU (metal/weights.rs:928-953)
-            check(lib().im_cuda_model_load_dense(self._model, name.encode(), vp(data), C.c_size_t(data.size)))
-            return
-        if len(t.shape) != 2:
-            raise InferenceError("Runtime", f"{name}: quantized tensor must be 2-D, got shape {t.shape}")
-        N, K = t.shape
-        sc, zp = np.ascontiguousarray(t.scale), np.ascontiguousarray(t.zero_point)
-        if sc.dtype != zp.dtype:
-            sc, zp = sc.astype(np.float32), zp.astype(np.float32)
-        pd = IM_DTYPE_F32 if sc.dtype == np.float32 else IM_DTYPE_F16
-        awq = None if t.awq_scales is None else np.ascontiguousarray(t.awq_scales, dtype=np.float16)
-        codes = np.ascontiguousarray(t.data, dtype=np.uint8)
-        check(lib().im_cuda_model_load_affine(self._model, name.encode(), vp(codes), vp(sc), vp(zp), C.c_int(pd), vp(awq),
-                                              C.c_int(N), C.c_int(K), C.c_int(t.group_size), C.c_int(t.bit_width)))
+        self._family.load_tensor(self._model, name, t)
 
     @_wrap
     def tp_init(self, unique_id: bytes) -> None:
@@ -246,6 +209,32 @@ class CudaInference:
         self._next = getattr(self, "_next", {})
         self._next[sid.value] = int(_argmax_last(out))
         return sid.value
+
+    @_wrap
+    def open_sequence(self) -> int:
+        """A free cache slot without tokens yet; extend_sequence() feeds it."""
+        self._need_model()
+        sid = C.c_int(-1)
+        check(lib().im_cuda_model_seq_open(self._model, C.byref(sid)))
+        return sid.value
+
+    @_wrap
+    def extend_sequence(self, seq_id: int, tokens, want=()) -> np.ndarray:
+        """More tokens for a live sequence, in a portion of any length; returns the logits [len(want), vocab] of the named
+        places among them (ascending).  A single token takes the captured decode step, like batch_decode_step."""
+        self._need_model()
+        toks = np.ascontiguousarray(tokens, dtype=np.uint32).reshape(-1)
+        want = np.ascontiguousarray(want, dtype=np.int32).reshape(-1)
+        if toks.size == 1 and self.sequence_position(seq_id) > 0:
+            if want.size > 1 or (want.size and want[0] != 0):
+                raise InferenceError("Runtime", "wanted place outside the portion")
+            out = np.empty((1, self._mc.vocab_size), dtype=np.float32)
+            ids = np.array([seq_id], dtype=np.int32)
+            check(lib().im_cuda_model_batch_decode_step(self._model, vp(ids), vp(toks), C.c_int(1), vp(out)))
+            return out[:want.size]
+        out = np.empty((want.size, self._mc.vocab_size), dtype=np.float32)
+        check(lib().im_cuda_model_seq_extend(self._model, C.c_int(seq_id), vp(toks), C.c_int(toks.size), vp(want), C.c_int(want.size), vp(out)))
+        return out
 
     @_wrap
     def remove_sequence(self, seq_id: int) -> None:
