@@ -1,7 +1,7 @@
 #!/usr/bin/env python
 """Benchmark of the quantized decode hot path on B200.
 
-    python bench.py [--gpus N] [--steps K] [--warmup W] [--impl reference] [--workload decode|matvec|attention]
+    python bench.py [--gpus N] [--steps K] [--warmup W] [--impl reference] [--workload decode|matvec|attention|stack]
                     [--prompt P] [--batch B]
 
 Prints ONE JSON line (rank 0).  Workloads are synthetic and seeded (random-init weights of the named
@@ -19,6 +19,11 @@ shape; no checkpoint or dataset is read):
           each step on a different weight copy out of a rotation larger than L2; value = GB/s.
 
   attention  TurboQuant INT8-KV decode attention alone at context --prompt and batch --batch (32 Q / 8 KV heads); GB/s of KV bytes.
+
+  stack   the Gizizen design at --stack-size (latent attention, latent attention, decayed linear attention, latent attention,
+          the first two looped three times: eight layer passes) with random bf16 weights, beside a Llama-shaped model of
+          this library with the same width, heads, feed-forward, vocabulary and number of passes (INT4 weights, fp16 KV):
+          prefill of --prompt tokens and greedy decode at --batch; value = decode tok/s of the former.
 
 `--impl reference` times the CPU restatement of the reference's own CPU path (the oracle) on the host
 cores for the same workload, on a bounded sample.
@@ -375,6 +380,139 @@ def run_decode(args, rank, world):
     if world == 1:
         out["cpu_baseline"] = cpu_decode_baseline(args.model, B, P, budget_s=20.0, min_steps=3)
     print(json.dumps(out))
+
+
+# ----------------------------------------------------------------------------- models given as a list of layers
+STACK_SIZES = {"w2048": dict(width=2048, ff=8192, heads=16, vocab=32768), "w4096": dict(width=4096, ff=14336, heads=32, vocab=32768)}
+
+
+def stack_model_json(size):
+    z = STACK_SIZES[size]
+    mlp = {"kind": "dense", "ff": z["ff"]}
+    lat = {"type": "latent_attention", "mlp": mlp,
+           "mixer": {"heads": z["heads"], "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5,
+                     "rot": {"dims": 64, "base": 5e5, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}}
+    lin = {"type": "lightning", "mlp": mlp,
+           "mixer": {"heads": z["heads"], "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-3 - 6 * i / z["heads"]) for i in range(z["heads"])]}}
+    return {"architecture": "Gizizen", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "layers": [lat, lat, lin, lat],
+            "loop": {"start": 0, "stop": 2, "times": 3}, "logit_softcap": 30.0}
+
+
+class SyntheticStackProvider:
+    """Random bf16 weights of a list-of-layers model, drawn on the GPU (rows scaled to keep activations near one)."""
+
+    def __init__(self, obj, seed=77):
+        from ironmill_b200.architectures import config_from_json
+        self.cfg, self.seed = config_from_json(obj), seed
+
+    def config(self):
+        return self.cfg
+
+    def has_tensor(self, name):
+        return name in self.cfg.tensors()
+
+    def tensor(self, name):
+        import zlib
+
+        import torch
+
+        from ironmill_b200.bundle import WeightTensor
+        shape = self.cfg.tensors()[name]
+        g = torch.Generator(device="cuda").manual_seed(self.seed * 7919 + zlib.crc32(name.encode()))
+        w = torch.ones(shape, device="cuda") if name.endswith(("norm", "norm1")) else torch.randn(shape, generator=g, device="cuda") * shape[-1] ** -0.5
+        return WeightTensor(w.to(torch.bfloat16).view(torch.uint16).cpu().numpy(), shape, "bfloat16")
+
+
+def stack_flops_per_token(cfg, ctx):
+    """Multiply-adds x 2 of one prompt token at mean context ctx: every projection, and attention in its expanded form
+    (the expansion of a token's keys and values once)."""
+    from ironmill_b200.stack_config import LatentAttention
+    order = list(range(cfg.loop_start)) + list(range(cfg.loop_start, cfg.loop_stop)) * cfg.loop_times + list(range(cfg.loop_stop, len(cfg.layers)))
+    w, n = cfg.hidden_size, 2 * cfg.hidden_size ** 2 * cfg.loop_times
+    for i in order:
+        L = cfg.layers[i]
+        m = L.mixer
+        n += 3 * w * L.ff + sum(a * b for a, b in (s for k, s in m.tensors(w).items() if len(s) == 2))
+        if isinstance(m, LatentAttention):
+            n += ctx * m.heads * (m.dim + m.rot_dim + m.vdim)
+        else:
+            n += 3 * m.heads * m.dim * m.vdim
+    return 2 * n
+
+
+def time_model(eng, vocab, P, B, K, W, reps=3):
+    """(prefill seconds per prompt, decode ms per step): prompts through add_sequence (host tokens in, last logits out),
+    then K greedy steps of B sequences timed with events on the engine's stream."""
+    import torch
+    prompt = np.random.Generator(np.random.PCG64(11)).integers(0, vocab, P).astype(np.uint32)
+    for _ in range(2):
+        eng.reset()
+        eng.prefill(prompt)
+    best = []
+    for _ in range(reps):
+        eng.reset()
+        torch.cuda.synchronize()
+        t0 = time.perf_counter()
+        lg = eng.prefill(prompt)
+        best.append(time.perf_counter() - t0)
+    eng.reset()
+    for _ in range(B):
+        eng.add_sequence(prompt)
+    toks, _ = eng.decode_greedy(np.full(B, int(lg.argmax()), np.uint32), W)
+    toks, ms = eng.decode_greedy(toks[-1], K)
+    return float(np.median(best)), ms / K
+
+
+def run_stack(args, rank, world):
+    import torch
+
+    from ironmill_b200 import ops
+    from ironmill_b200.bundle import ModelConfig
+    from ironmill_b200.engine import CudaConfig, CudaInference
+    if rank != 0:
+        return
+    torch.cuda.set_device(0)
+    B, P, K, W = args.batch, args.prompt, args.steps, max(args.warmup, 3)
+    z = STACK_SIZES[args.stack_size]
+    peak, peak_src = measured_peaks()
+    tpeak = measured_tensor_peak()
+    max_seq = P + W + K + 64
+    ours_p = SyntheticStackProvider(stack_model_json(args.stack_size))
+    cfg = ours_p.cfg
+    passes = len(cfg.layers) + (cfg.loop_stop - cfg.loop_start) * (cfg.loop_times - 1)
+    res, clocks = {}, None
+    which = ("stack", "blocks") if args.stack_arm == "both" else (args.stack_arm,)
+    for arm in which:
+        if arm == "stack":
+            eng = CudaInference(CudaConfig(max_seq_len=max_seq, max_batch=B))
+            eng.load_weights(ours_p)
+            flops = stack_flops_per_token(cfg, P / 2) * P
+        else:
+            mc = ModelConfig(**dict(L8, hidden_size=z["width"], intermediate_size=z["ff"], num_attention_heads=z["heads"], vocab_size=z["vocab"],
+                                    num_hidden_layers=passes))
+            eng = CudaInference(CudaConfig(max_seq_len=max_seq, max_batch=B).without_turboquant())
+            eng.load_weights(SyntheticL8Provider(mc, ops.Device(0)))
+            hd, h = 128, z["heads"]
+            flops = 2 * P * passes * (z["width"] * (2 * h * hd + 2 * 8 * hd + 3 * z["ff"]) + P / 2 * h * 2 * hd)
+        sampler = ClockSampler(0)
+        sampler.start()
+        pre_s, ms = time_model(eng, z["vocab"], P, B, K, W)
+        seen = sampler.stop()
+        clocks = clocks or seen
+        nbytes = eng.step_bytes(P + W + K // 2, B)
+        res[arm] = {"prefill_ms": round(pre_s * 1e3, 3), "prefill_tok_s": round(P / pre_s, 1), "prefill_tflops": round(flops / pre_s / 1e12, 1),
+                    "prefill_frac_of_bf16_peak": round(flops / pre_s / 1e12 / tpeak, 4), "decode_ms_per_step": round(ms, 4),
+                    "decode_tok_s": round(B * 1e3 / ms, 1), "decode_bytes_per_step": nbytes, "decode_gbs": round(nbytes / ms / 1e6, 1),
+                    "decode_frac_of_hbm": round(nbytes / ms / 1e6 / peak, 4), "launches_per_step": eng.step_launches(),
+                    "profile_ms": {k: round(v, 4) for k, v in eng.profile_step(B).items() if v}}
+        eng.close()
+    first = res[which[0]]
+    print(json.dumps({
+        "metric": "decode tok/s (list-of-layers model, bf16)", "value": first["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": K, "warmup": W,
+        "ms_per_step": first["decode_ms_per_step"], "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+        "config": dict(z, workload="stack", size=args.stack_size, layer_passes=passes, batch=B, prompt_tokens=P,
+                       l2_policy="inputs larger than L2: every step streams all weights"),
+        "arms": res, "peaks": {"hbm_gbs": peak, "bf16_tflops": tpeak, "source": peak_src}, "clocks": clocks}))
 
 
 def decode_config(workload, cfg, B, P, world):
@@ -780,13 +918,15 @@ def main():
     ap.add_argument("--steps", type=int, default=256)
     ap.add_argument("--warmup", type=int, default=16)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="decode", choices=["decode", "matvec", "attention"])
+    ap.add_argument("--workload", default="decode", choices=["decode", "matvec", "attention", "stack"])
     ap.add_argument("--prompt", type=int, default=2048)
     ap.add_argument("--batch", type=int, default=1)
     ap.add_argument("--layers", type=int, default=0, help="decoder layers of the synthetic model (0 = the named model's; fewer only for profiler captures)")
     ap.add_argument("--sweep", type=int, default=1, help="matvec workload: 1 = also time every shape at batch 1/4/16/64, INT8 and the tensor-parallel shards")
     ap.add_argument("--kv-bits", type=int, default=8, choices=[4, 8, 16], help="attention workload: TurboQuant bits, or 16 = fp16 KV cache")
     ap.add_argument("--model", default="llama3_8b", choices=sorted(MODELS), help="decode workload shape (the default is the headline configuration)")
+    ap.add_argument("--stack-size", default="w2048", choices=sorted(STACK_SIZES), help="stack workload: sizes of the model")
+    ap.add_argument("--stack-arm", default="both", choices=["both", "stack", "blocks"], help="stack workload: only the list-of-layers model, or only its Llama-shaped counterpart")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", 0))
     world = int(os.environ.get("WORLD_SIZE", 1))
@@ -796,6 +936,8 @@ def main():
         run_matvec(args, rank, world)
     elif args.workload == "attention":
         run_attention(args, rank, world)
+    elif args.workload == "stack":
+        run_stack(args, rank, world)
     else:
         run_decode(args, rank, world)
     import torch.distributed as dist
