@@ -90,16 +90,18 @@ __global__ void __launch_bounds__(kMvThreads, NB <= 4 ? 2 : 1) dense_matvec_kern
     const int kv = w.ld / V, nit = (kv + 32 * kMvU * KS - 1) / (32 * kMvU * KS);
     const int ntiles = (w.N + 2 * groups - 1) / (2 * groups);
     const T *W = static_cast<const T *>(w.w);
-    uint4 nxt[2][kMvU];
+    uint4 nxt[2][kMvU] = {};
+    // Every address is clamped into the matrix (rows past the end repeat the last one, columns past the end the last
+    // vector): the streaming load is inline assembly without side effects, which a compiler may move above a guard.
     auto load = [&](int tile, int it) {
+        if (tile >= ntiles) return;
         const int n0 = (tile * groups + grp) * 2;
 #pragma unroll
-        for (int r = 0; r < 2; r++)
+        for (int r = 0; r < 2; r++) {
+            const T *row = W + (size_t)min(n0 + r, w.N - 1) * w.ld;
 #pragma unroll
-            for (int u = 0; u < kMvU; u++) {
-                const int i = ((it * KS + ks) * kMvU + u) * 32 + lane;
-                nxt[r][u] = (tile < ntiles && n0 + r < w.N && i < kv) ? ldg_stream_v4(W + (size_t)(n0 + r) * w.ld + (size_t)i * V) : make_uint4(0, 0, 0, 0);
-            }
+            for (int u = 0; u < kMvU; u++) nxt[r][u] = ldg_stream_v4(row + (size_t)min(((it * KS + ks) * kMvU + u) * 32 + lane, kv - 1) * V);
+        }
     };
     pdl_trigger();
     load(blockIdx.x, 0);  // weights are constants: requested before the predecessor has finished
@@ -118,7 +120,7 @@ __global__ void __launch_bounds__(kMvThreads, NB <= 4 ? 2 : 1) dense_matvec_kern
 #pragma unroll
                 for (int u = 0; u < kMvU; u++) cur[r][u] = nxt[r][u];
             if (it + 1 < nit) load(tile, it + 1);
-            else load(tile + gridDim.x, 0);
+            else load(tile + (int)gridDim.x, 0);
 #pragma unroll
             for (int u = 0; u < kMvU; u++) {
                 const int i = ((it * KS + ks) * kMvU + u) * 32 + lane;
