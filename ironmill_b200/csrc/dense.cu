@@ -182,12 +182,18 @@ __global__ void __launch_bounds__(256) dense_stage_kernel(const DenseSrc src, in
 }
 
 // ---- tcgen05 GEMM ----------------------------------------------------------------------------------------------------
+// Persistent: a CTA walks work items (weight tile, token tile, K slice), token tiles of one weight tile next to each other
+// so that the weights stream from memory once.  Two accumulators in tensor memory: the epilogue warps convert and store one
+// item while the next one's products run.
 constexpr int kDM = 128, kDK = 64;  // weight rows and columns of a stage (one 128-byte swizzle row)
-constexpr int kDThreads = 192;      // warps 0-3: epilogue, 4: copies, 5: tensor memory + MMA issue
+constexpr int kDEpi = 8;            // epilogue warps: warp w reads tensor-memory lanes 32 (w % 4) .., half w / 4 of the tokens
+constexpr int kDThreads = (kDEpi + 2) * 32;  // ... then one warp for the copies, one for tensor memory + MMA issue
 template <int TN>
 constexpr int dense_stages() { return TN >= 256 ? 4 : TN == 128 ? 3 : 4; }
 template <int TN>
-constexpr int dense_gemm_smem() { return 1024 + dense_stages<TN>() * (kDM * 128 + TN * 128) + (2 * dense_stages<TN>() + 1) * 8 + 16; }
+constexpr int dense_gemm_smem() { return 1024 + dense_stages<TN>() * (kDM * 128 + TN * 128) + (2 * dense_stages<TN>() + 4) * 8 + 16; }
+template <int TN>
+constexpr int dense_ctas_per_sm() { return TN >= 256 ? 1 : 2; }
 
 __device__ __forceinline__ uint64_t dense_desc_sw128(uint32_t smem_addr) {
     // K-major, 128-byte swizzle: start >> 4, leading offset 1, stride offset 1024 B >> 4, version 1, layout 2 (see gemm_tc.cu)
@@ -202,17 +208,17 @@ __device__ __forceinline__ void dense_mma(uint32_t tmem_d, uint64_t a, uint64_t 
 __device__ __forceinline__ void dense_commit(uint64_t *bar) {
     asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(smem_u32(bar)) : "memory");
 }
-__device__ __forceinline__ void dense_tmem_ld32(uint32_t taddr, uint32_t (&r)[32]) {
+__device__ __forceinline__ void dense_tmem_ld16(uint32_t taddr, float (&v)[16]) {
+    uint32_t r[16];
     asm volatile(
-        "tcgen05.ld.sync.aligned.32x32b.x32.b32"
-        "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15,"
-        " %16, %17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31}, [%32];\n"
+        "tcgen05.ld.sync.aligned.32x32b.x16.b32"
+        "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];\n"
         : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]),
-          "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]), "=r"(r[17]), "=r"(r[18]),
-          "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]),
-          "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
+          "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
         : "r"(taddr));
     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+#pragma unroll
+    for (int i = 0; i < 16; i++) v[i] = __uint_as_float(r[i]);
 }
 __device__ __forceinline__ void dense_tma_2d(void *dst, const CUtensorMap *map, int x, int y, uint64_t *bar) {
     // x is a multiple of 64 elements (128 bytes)
@@ -220,38 +226,108 @@ __device__ __forceinline__ void dense_tma_2d(void *dst, const CUtensorMap *map, 
                  "r"(x), "r"(y), "r"(smem_u32(bar))
                  : "memory");
 }
+// bf16 epilogues: z sigmoid(z), and gelu_tanh(z) = z / (1 + exp(-2 u)), u = sqrt(2 / pi) (z + 0.044715 z^3); the error of the
+// fast exponential and quotient (about 1e-6) is far below the bf16 result's rounding
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
+__device__ __forceinline__ float gelu_mul_fast(float z, float up) {
+    const float w = -1.5957691216057308f * z * fmaf(0.044715f * z, z, 1.0f);
+    return __fdividef(z * up, 1.0f + __expf(fminf(w, 80.0f)));
+}
 
 struct DenseGemm {
     int N, M, kblocks, kb_per;  // kblocks: 64-column blocks of K; kb_per: of one K slice
+    int mtiles, ntiles, slices;
     float *partial;             // [slices][M][N] when K is split
     int *err;
     DenseEpi epi;
 };
 
-// D[128 weight rows x TN tokens] += W[128 x 64] X[TN x 64]^T per stage; grid (row tiles, token tiles, K slices).
-template <int TN>
-__global__ void __launch_bounds__(kDThreads) dense_gemm_tc_kernel(const DenseGemm p, const __grid_constant__ CUtensorMap ta, const __grid_constant__ CUtensorMap tb) {
+// 16 tokens m .. m + 15 of row n (one per lane) of the f32 sums
+__device__ __forceinline__ void dense_store16(const DenseGemm &p, int z, int n, int n_warp, int m, const float (&v)[16]) {
     typedef __nv_bfloat16 T;
+    const DenseEpi &e = p.epi;
+    const int lane = threadIdx.x & 31, left = p.M - m;
+    if (p.partial) {
+        if (n < p.N) {
+            float *dst = p.partial + ((size_t)z * p.M + m) * p.N + n;
+#pragma unroll
+            for (int i = 0; i < 16; i++)
+                if (i < left) dst[(size_t)i * p.N] = v[i];
+        }
+    } else if (e.kind == kEpiProj) {
+        if (n_warp + 31 >= e.pair0) {
+            // (gate, up) sit in neighbouring lanes: of two tokens, the even lane takes the first, the odd lane the second
+            // (pair0 is a multiple of eight: no pair straddles it)
+            T *act = static_cast<T *>(e.act) + (size_t)m * e.ldact + ((n - e.pair0) >> 1);
+            T *y = static_cast<T *>(e.y) + (size_t)m * e.ldy + n;
+            const bool odd = lane & 1, pair = n >= e.pair0;
+#pragma unroll
+            for (int i = 0; i < 16; i += 2) {
+                const float got = __shfl_xor_sync(0xffffffffu, odd ? v[i] : v[i + 1], 1);
+                if (pair) {
+                    const float r = odd ? gelu_mul_fast(got, v[i + 1]) : gelu_mul_fast(v[i], got);
+                    if (n < p.N && i + odd < left) act[(size_t)(i + odd) * e.ldact] = from_f<T>(r);
+                } else {
+#pragma unroll
+                    for (int j = 0; j < 2; j++)
+                        if (i + j < left) y[(size_t)(i + j) * e.ldy] = from_f<T>(n < e.silu_end ? silu_fast(v[i + j]) : v[i + j]);
+                }
+            }
+        } else {
+            T *y = static_cast<T *>(e.y) + (size_t)m * e.ldy + n;
+            const bool act = n < e.silu_end;
+            if (n < p.N)
+#pragma unroll
+                for (int i = 0; i < 16; i++)
+                    if (i < left) y[(size_t)i * e.ldy] = from_f<T>(act ? silu_fast(v[i]) : v[i]);
+        }
+    } else if (n < p.N) {
+        float *x = e.xf + (size_t)m * e.ldx + n;
+        if (e.kind == kEpiResidual) {
+            float old[16];
+#pragma unroll
+            for (int i = 0; i < 16; i++) old[i] = i < left ? x[(size_t)i * e.ldx] : 0.0f;
+#pragma unroll
+            for (int i = 0; i < 16; i++)
+                if (i < left) x[(size_t)i * e.ldx] = old[i] + v[i];
+        } else {
+            const float b = e.bias ? e.bias[n] : 0.0f;
+#pragma unroll
+            for (int i = 0; i < 16; i++) {
+                float r = v[i] + b;
+                if (e.cap > 0.0f) r = e.cap * tanhf(r / e.cap);
+                if (i < left) x[(size_t)i * e.ldx] = r;
+            }
+        }
+    }
+}
+
+// D[128 weight rows x TN tokens] += W[128 x 64] X[TN x 64]^T per stage.
+template <int TN>
+__global__ void __launch_bounds__(kDThreads, dense_ctas_per_sm<TN>()) dense_gemm_tc_kernel(const DenseGemm p, const __grid_constant__ CUtensorMap ta,
+                                                                                         const __grid_constant__ CUtensorMap tb) {
     constexpr int S = dense_stages<TN>();
-    constexpr int kA = kDM * 128, kB = TN * 128;
+    constexpr int kA = kDM * 128, kB = TN * 128, kCols = 2 * TN;
     extern __shared__ __align__(1024) unsigned char dense_gemm_raw[];
     unsigned char *smem = reinterpret_cast<unsigned char *>((reinterpret_cast<uintptr_t>(dense_gemm_raw) + 1023) & ~(uintptr_t)1023);
     unsigned char *As = smem, *Bs = smem + S * kA;
-    uint64_t *full = reinterpret_cast<uint64_t *>(Bs + S * kB), *empty = full + S, *accum = empty + S;
-    uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(accum + 1);
+    uint64_t *full = reinterpret_cast<uint64_t *>(Bs + S * kB), *empty = full + S, *tfull = empty + S, *tempty = tfull + 2;
+    uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(tempty + 2);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int n0 = blockIdx.x * kDM, m0 = blockIdx.y * TN;
     pdl_trigger();
     if (tid == 0) {
         for (int i = 0; i < S; i++) {
             mbar_init(&full[i], 1);
             mbar_init(&empty[i], 1);
         }
-        mbar_init(accum, 1);
+        for (int i = 0; i < 2; i++) {
+            mbar_init(&tfull[i], 1);
+            mbar_init(&tempty[i], kDEpi);
+        }
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
-    if (warp == 5) {
-        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(tmem_slot)), "r"(TN < 32 ? 32 : TN) : "memory");
+    if (warp == kDEpi + 1) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(tmem_slot)), "r"(kCols) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -259,98 +335,74 @@ __global__ void __launch_bounds__(kDThreads) dense_gemm_tc_kernel(const DenseGem
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const uint32_t tmem_d = *tmem_slot;
     pdl_wait();
-    const int kb0 = blockIdx.z * p.kb_per, nkb = min(p.kblocks, kb0 + p.kb_per) - kb0;
+    const int items = p.mtiles * p.ntiles * p.slices;
     bool ok = true;
-    if (warp == 4) {
-        for (int it = 0; it < nkb; it++) {
-            const int s = it % S, use = it / S;
-            if (ok && use > 0 && !mbar_wait_warp(&empty[s], (use - 1) & 1, p.err)) ok = false;
-            if (lane == 0 && ok) {
-                mbar_expect_tx(&full[s], (uint32_t)(kA + kB));
-                dense_tma_2d(As + (size_t)s * kA, &ta, (kb0 + it) * kDK, n0, &full[s]);
-                dense_tma_2d(Bs + (size_t)s * kB, &tb, (kb0 + it) * kDK, m0, &full[s]);
+    if (warp == kDEpi) {
+        int it = 0;
+        for (int w = blockIdx.x; w < items; w += gridDim.x) {
+            const int m0 = w % p.mtiles * TN, n0 = w / p.mtiles % p.ntiles * kDM, kb0 = w / (p.mtiles * p.ntiles) * p.kb_per;
+            const int kb1 = min(p.kblocks, kb0 + p.kb_per);
+            for (int kb = kb0; kb < kb1; kb++, it++) {
+                const int s = it % S, use = it / S;
+                if (ok && use > 0 && !mbar_wait_warp(&empty[s], (use - 1) & 1, p.err)) ok = false;
+                if (lane == 0 && ok) {
+                    mbar_expect_tx(&full[s], (uint32_t)(kA + kB));
+                    dense_tma_2d(As + (size_t)s * kA, &ta, kb * kDK, n0, &full[s]);
+                    dense_tma_2d(Bs + (size_t)s * kB, &tb, kb * kDK, m0, &full[s]);
+                }
+                __syncwarp();
             }
-            __syncwarp();
         }
-    } else if (warp == 5) {
+    } else if (warp == kDEpi + 1) {
         // f32 accumulator, bf16 operands, both K-major, N >> 3 in bits 17-22, M >> 4 in bits 24-28
         constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(TN >> 3) << 17) | ((uint32_t)(kDM >> 4) << 24);
-        for (int it = 0; it < nkb; it++) {
-            const int s = it % S, use = it / S;
-            if (ok && !mbar_wait_warp(&full[s], use & 1, p.err)) ok = false;
+        int it = 0, cnt = 0;
+        for (int w = blockIdx.x; w < items; w += gridDim.x, cnt++) {
+            const int kb0 = w / (p.mtiles * p.ntiles) * p.kb_per, kb1 = min(p.kblocks, kb0 + p.kb_per);
+            const int acc = cnt & 1, use = cnt >> 1;
+            if (ok && use > 0 && !mbar_wait_warp(&tempty[acc], (use - 1) & 1, p.err)) ok = false;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            if (lane == 0 && ok) {
-                const uint32_t a0 = smem_u32(As + (size_t)s * kA), b0 = smem_u32(Bs + (size_t)s * kB);
+            for (int kb = kb0; kb < kb1; kb++, it++) {
+                const int s = it % S;
+                if (ok && !mbar_wait_warp(&full[s], (it / S) & 1, p.err)) ok = false;
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                if (lane == 0 && ok) {
+                    const uint32_t a0 = smem_u32(As + (size_t)s * kA), b0 = smem_u32(Bs + (size_t)s * kB);
 #pragma unroll
-                for (int j = 0; j < 4; j++)
-                    dense_mma(tmem_d, dense_desc_sw128(a0 + j * 32), dense_desc_sw128(b0 + j * 32), idesc, (it > 0 || j > 0) ? 1u : 0u);
-                dense_commit(&empty[s]);
-                if (it == nkb - 1) dense_commit(accum);
+                    for (int j = 0; j < 4; j++)
+                        dense_mma(tmem_d + (uint32_t)(acc * TN), dense_desc_sw128(a0 + j * 32), dense_desc_sw128(b0 + j * 32), idesc, (kb > kb0 || j > 0) ? 1u : 0u);
+                    dense_commit(&empty[s]);
+                    if (kb == kb1 - 1) dense_commit(&tfull[acc]);
+                }
+                __syncwarp();
             }
-            __syncwarp();
         }
     } else {
-        if (!mbar_wait_warp(accum, 0, p.err)) ok = false;
-        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        const int n = n0 + tid;  // this thread's tensor-memory lane
-        if (ok) {
+        int cnt = 0;
+        for (int w = blockIdx.x; w < items; w += gridDim.x, cnt++) {
+            const int m0 = w % p.mtiles * TN, n_warp = w / p.mtiles % p.ntiles * kDM + (warp & 3) * 32, z = w / (p.mtiles * p.ntiles);
+            const int acc = cnt & 1;
+            if (ok && !mbar_wait_warp(&tfull[acc], (cnt >> 1) & 1, p.err)) ok = false;
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            if (ok) {
+                const int c_begin = (warp >> 2) * (TN / 2);
 #pragma unroll 1
-            for (int c0 = 0; c0 < TN && m0 + c0 < p.M; c0 += 32) {
-                uint32_t r[32];
-                dense_tmem_ld32(tmem_d + ((uint32_t)(warp * 32) << 16) + (uint32_t)c0, r);
-                if (p.partial) {
-                    if (n < p.N) {
-                        float *dst = p.partial + (size_t)blockIdx.z * p.M * p.N + n;
-#pragma unroll
-                        for (int i = 0; i < 32; i++)
-                            if (m0 + c0 + i < p.M) dst[(size_t)(m0 + c0 + i) * p.N] = __uint_as_float(r[i]);
-                    }
-                } else if (p.epi.kind == kEpiProj) {
-                    if (n0 + warp * 32 + 31 >= p.epi.pair0) {  // pairs in this warp (pair0 is even: a pair never straddles)
-#pragma unroll
-                        for (int i = 0; i < 32; i++) {
-                            const float v = __uint_as_float(r[i]), o = __shfl_xor_sync(0xffffffffu, v, 1);
-                            const int m = m0 + c0 + i;
-                            if (m < p.M && n < p.N && !(lane & 1)) epi_pair<T>(p.epi, m, n, v, o, p.N);
-                        }
-                    } else {
-                        T *y = static_cast<T *>(p.epi.y) + n;
-                        const bool act = n < p.epi.silu_end;
-#pragma unroll
-                        for (int i = 0; i < 32; i++) {
-                            const int m = m0 + c0 + i;
-                            float v = __uint_as_float(r[i]);
-                            if (act) v = silu_f(v);
-                            if (m < p.M && n < p.N) y[(size_t)m * p.epi.ldy] = from_f<T>(v);
-                        }
-                    }
-                } else if (n < p.N) {
-                    float *x = p.epi.xf + n;
-                    if (p.epi.kind == kEpiResidual) {
-                        float old[32];
-#pragma unroll
-                        for (int i = 0; i < 32; i++) old[i] = m0 + c0 + i < p.M ? x[(size_t)(m0 + c0 + i) * p.epi.ldx] : 0.0f;
-#pragma unroll
-                        for (int i = 0; i < 32; i++)
-                            if (m0 + c0 + i < p.M) x[(size_t)(m0 + c0 + i) * p.epi.ldx] = old[i] + __uint_as_float(r[i]);
-                    } else {
-                        const float b = p.epi.bias ? p.epi.bias[n] : 0.0f;
-#pragma unroll
-                        for (int i = 0; i < 32; i++) {
-                            float v = __uint_as_float(r[i]) + b;
-                            if (p.epi.cap > 0.0f) v = p.epi.cap * tanhf(v / p.epi.cap);
-                            if (m0 + c0 + i < p.M) x[(size_t)(m0 + c0 + i) * p.epi.ldx] = v;
-                        }
-                    }
+                for (int c = c_begin; c < c_begin + TN / 2 && m0 + c < p.M; c += 16) {
+                    float v[16];
+                    dense_tmem_ld16(tmem_d + ((uint32_t)((warp & 3) * 32) << 16) + (uint32_t)(acc * TN + c), v);
+                    dense_store16(p, z, n_warp + lane, n_warp, m0 + c, v);
                 }
             }
+            asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&tempty[acc]);
         }
     }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
     __syncthreads();
-    if (warp == 5) {
+    if (warp == kDEpi + 1) {
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_d), "r"(TN < 32 ? 32 : TN) : "memory");
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_d), "r"(kCols) : "memory");
     }
 }
 
@@ -456,14 +508,17 @@ int bf16_tmap(const void *base, int rows, int cols, int ld, int box_rows, CUtens
 }
 
 template <int TN>
-int gemm_launch(DenseGemm p, const DenseWeight &w, const void *x, int ldx, int slices, cudaStream_t st) {
+int gemm_launch(const Device *dev, DenseGemm p, const DenseWeight &w, const void *x, int ldx, int slices, cudaStream_t st) {
     alignas(64) CUtensorMap ta, tb;
     int rc = bf16_tmap(w.w, w.N, w.K, w.ld, kDM, &ta);
     if (rc != IM_OK) return rc;
     rc = bf16_tmap(x, p.M, w.K, ldx, TN, &tb);
     if (rc != IM_OK) return rc;
-    IM_CUDA_CHECK(launch_k(dense_gemm_tc_kernel<TN>, dim3((p.N + kDM - 1) / kDM, (p.M + TN - 1) / TN, slices), dim3(kDThreads), (size_t)dense_gemm_smem<TN>(), st, p,
-                           ta, tb));
+    p.mtiles = (p.M + TN - 1) / TN;
+    p.ntiles = (p.N + kDM - 1) / kDM;
+    p.slices = slices;
+    const int ctas = std::min(p.mtiles * p.ntiles * slices, dev->sm_count * dense_ctas_per_sm<TN>());
+    IM_CUDA_CHECK(launch_k(dense_gemm_tc_kernel<TN>, dim3(ctas), dim3(kDThreads), (size_t)dense_gemm_smem<TN>(), st, p, ta, tb));
     if (p.partial) {
         const size_t n = (size_t)p.M * ((p.N + 1) / 2);
         IM_CUDA_CHECK(launch_k(dense_splitk_reduce_kernel<__nv_bfloat16>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, st, (const float *)p.partial, p.epi, p.M, p.N,
@@ -556,10 +611,10 @@ int dense_project(const Device *dev, const DenseWeight &w, const DenseSrc &src, 
         }
     }
     const long long ctas256 = (long long)tiles * ((M + 255) / 256);
-    if (M > 128 && ctas256 >= dev->sm_count) return gemm_launch<256>(p, w, x, ldx, slices, st);
-    if (M > 64) return gemm_launch<128>(p, w, x, ldx, slices, st);
-    if (M > 32) return gemm_launch<64>(p, w, x, ldx, slices, st);
-    return gemm_launch<32>(p, w, x, ldx, slices, st);
+    if (M > 128 && ctas256 >= dev->sm_count) return gemm_launch<256>(dev, p, w, x, ldx, slices, st);
+    if (M > 64) return gemm_launch<128>(dev, p, w, x, ldx, slices, st);
+    if (M > 32) return gemm_launch<64>(dev, p, w, x, ldx, slices, st);
+    return gemm_launch<32>(dev, p, w, x, ldx, slices, st);
 }
 
 int stack_embed(const uint32_t *tokens, const void *table, int f32, int ld, const float *gamma, float *x, float *x0, int width, uint32_t vocab, float eps, int M,

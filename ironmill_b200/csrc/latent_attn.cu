@@ -457,20 +457,37 @@ __device__ __forceinline__ float row_norm(const LatentPart &p, size_t row, float
     return 1.0f / l;
 }
 
-// grid (rows, column blocks of 128): the splits of a row added up and normalised, into the row's first split
+// grid (rows, column blocks of 128): the splits of a row added up and normalised
 __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentPart p, const float *__restrict__ sink, int heads, int latP, float *__restrict__ out) {
+    __shared__ float wk[256], sm[4], sl[4];
+    const size_t row = blockIdx.x;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const float s = sink ? sink[row % heads] : -INFINITY;
     pdl_trigger();
     pdl_wait();
-    __shared__ float wk[256];
-    const size_t row = blockIdx.x;
-    float gm;
-    const float inv = row_norm(p, row, sink ? sink[row % heads] : -INFINITY, &gm);
-    for (int k = threadIdx.x; k < p.splits; k += 128) {
-        const float m = p.pm[row * p.splits + k];
-        wk[k] = m == -INFINITY ? 0.0f : expf(m - gm) * inv;
+    float m[2], l[2];
+#pragma unroll
+    for (int i = 0; i < 2; i++) {
+        const int k = tid + 128 * i;
+        m[i] = k < p.splits ? p.pm[row * p.splits + k] : -INFINITY;
+        l[i] = k < p.splits ? p.pl[row * p.splits + k] : 0.0f;
     }
+    float gm = warp_max(fmaxf(m[0], m[1]));
+    if (lane == 0) sm[warp] = gm;
     __syncthreads();
-    const int c = blockIdx.y * 128 + threadIdx.x;
+    gm = fmaxf(fmaxf(fmaxf(sm[0], sm[1]), fmaxf(sm[2], sm[3])), s);
+    float sum = 0.0f;
+#pragma unroll
+    for (int i = 0; i < 2; i++) {
+        m[i] = m[i] == -INFINITY ? 0.0f : expf(m[i] - gm);
+        wk[tid + 128 * i] = m[i];
+        sum = fmaf(l[i], m[i], sum);
+    }
+    sum = warp_sum(sum);
+    if (lane == 0) sl[warp] = sum;
+    __syncthreads();
+    const float inv = 1.0f / (sl[0] + sl[1] + sl[2] + sl[3] + (s == -INFINITY ? 0.0f : expf(s - gm)));
+    const int c = blockIdx.y * 128 + tid;
     if (c >= latP) return;
     float acc = 0.0f;
 #pragma unroll 8
@@ -478,7 +495,7 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentPart p,
         const float w = wk[k];
         if (w != 0.0f) acc = fmaf(w, p.po[(row * p.splits + k) * latP + c], acc);
     }
-    out[row * latP + c] = acc;
+    out[row * latP + c] = acc * inv;
 }
 
 // grid (heads, slices of the value rows, token groups of MB): out[m, h] = W_uv[h] o'.  src: the normalised sums, or (single
@@ -526,14 +543,14 @@ __global__ void __launch_bounds__(256) latent_out_kernel(const LatentArgs a, con
 }
 
 // ---- expanded form ------------------------------------------------------------------------------------------------------
-// grid (ceil(T / 128), heads of the group), 8 warps of 16 tokens.  K tile: [expanded key | rotated part of the cache row].
-constexpr int kLpM = 128, kLpN = 64;
+// grid (ceil(T / 64), heads of the group), 4 warps of 16 tokens, three such CTAs per SM.  K tile: [expanded key | rotated part of the cache row].
+constexpr int kLpM = 64, kLpN = 32, kLpThreads = kLpM * 2, kLpNB = kLpN / 8;
 inline int prefill_qk(const LatentShape &s) { return round_up(s.dimP + s.rotP, 32); }
 inline size_t latent_prefill_smem(const LatentShape &s, int dv) { return (size_t)(kLpM + 2 * kLpN) * (prefill_qk(s) + 8) * 2 + (size_t)2 * kLpN * (dv + 8) * 2; }
 
 template <int DV>  // value columns, padded
-__global__ void __launch_bounds__(256, 1) latent_prefill_kernel(const LatentArgs a, const __nv_bfloat16 *__restrict__ kv, int ldkv, int h0, int qk) {
-    constexpr int NT = 256, ND = DV / 8;
+__global__ void __launch_bounds__(kLpThreads, DV <= 128 ? 3 : 1) latent_prefill_kernel(const LatentArgs a, const __nv_bfloat16 *__restrict__ kv, int ldkv, int h0, int qk) {
+    constexpr int NT = kLpThreads, ND = DV / 8;
     extern __shared__ __align__(16) unsigned char latent_smem[];
     const LatentShape &s = a.s;
     const int rs = (qk + 8) * 2, vs = (DV + 8) * 2;
@@ -590,16 +607,16 @@ __global__ void __launch_bounds__(256, 1) latent_prefill_kernel(const LatentArgs
         }
         __syncthreads();
         if (p0 < warp_end) {
-            float sc[8][4];
+            float sc[kLpNB][4];
 #pragma unroll
-            for (int nb = 0; nb < 8; nb++) sc[nb][0] = sc[nb][1] = sc[nb][2] = sc[nb][3] = 0.0f;
+            for (int nb = 0; nb < kLpNB; nb++) sc[nb][0] = sc[nb][1] = sc[nb][2] = sc[nb][3] = 0.0f;
 #pragma unroll 2
             for (int kk = 0; kk < qk / 32; kk++) {
                 unsigned a0[4], a1[4];
                 ldsm_x4(a0, qa + kk * 64);
                 ldsm_x4(a1, qa + kk * 64 + 32);
 #pragma unroll
-                for (int nb = 0; nb < 8; nb++) {
+                for (int nb = 0; nb < kLpNB; nb++) {
                     unsigned b[4];
                     ldsm_x4(b, ka + (buf * kLpN + 8 * nb) * rs + kk * 64);
                     mma_bf16(sc[nb], a0[0], a0[1], a0[2], a0[3], b[0], b[1]);
@@ -608,7 +625,7 @@ __global__ void __launch_bounds__(256, 1) latent_prefill_kernel(const LatentArgs
             }
             float corr[2], mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
-            for (int nb = 0; nb < 8; nb++)
+            for (int nb = 0; nb < kLpNB; nb++)
 #pragma unroll
                 for (int e = 0; e < 4; e++) {
                     const int p = p0 + 8 * nb + 2 * t + (e & 1);
@@ -630,7 +647,7 @@ __global__ void __launch_bounds__(256, 1) latent_prefill_kernel(const LatentArgs
                 o[i][2] *= corr[1]; o[i][3] *= corr[1];
             }
 #pragma unroll
-            for (int kb = 0; kb < 4; kb++) {
+            for (int kb = 0; kb < kLpN / 16; kb++) {
                 unsigned hi[4], lo[4];
 #pragma unroll
                 for (int hb = 0; hb < 2; hb++)
@@ -732,7 +749,7 @@ int out_launch(const LatentArgs &a, const LatentPart &p, const float *src, int n
 
 template <int DV>
 int prefill_launch(const LatentArgs &a, const __nv_bfloat16 *kv, int ldkv, int h0, int nh, cudaStream_t st) {
-    IM_CUDA_CHECK(launch_k(latent_prefill_kernel<DV>, dim3((a.T + kLpM - 1) / kLpM, nh), dim3(256), latent_prefill_smem(a.s, DV), st, a, kv, ldkv, h0, prefill_qk(a.s)));
+    IM_CUDA_CHECK(launch_k(latent_prefill_kernel<DV>, dim3((a.T + kLpM - 1) / kLpM, nh), dim3(kLpThreads), latent_prefill_smem(a.s, DV), st, a, kv, ldkv, h0, prefill_qk(a.s)));
     return IM_OK;
 }
 int prefill_dv(const LatentShape &s) { return s.vP <= 32 ? 32 : s.vP <= 64 ? 64 : s.vP <= 128 ? 128 : s.vP <= 256 ? 256 : 0; }

@@ -86,9 +86,17 @@ inline size_t linear_chunk_smem(int C, int dimK, int bufs) {
     return (size_t)bufs * C * (2 * (dimK + 8) * 2 + kLcRow) + 3 * (size_t)C * kLcRow + 3 * (size_t)dimK * kLcRow + (size_t)(C + 1) * 4;
 }
 
-// grid (column blocks of 32, heads, sequences), C / 16 warps.  MW: 16-row tiles of the state per warp.
+// A long prompt of one sequence is cut into segments that run side by side: a first pass (`local`) leaves what each segment
+// but the last adds to a zero state, the second starts every segment from the state those sums make before it.
+struct LinearSegments {
+    int count = 1, tokens = 0;  // segments, tokens of each (a multiple of kLinearPow)
+    int local = 0;
+    float *sums = nullptr;      // [count - 1][heads][dim][vdim]
+};
+
+// grid (column blocks of 32, heads, sequences or segments), C / 16 warps.  MW: 16-row tiles of the state per warp.
 template <int C, int MW>
-__global__ void __launch_bounds__(C * 2, 1) linear_chunk_kernel(const LinearArgs a, int dimK, int bufs) {
+__global__ void __launch_bounds__(C * 2, 1) linear_chunk_kernel(const LinearArgs a, int dimK, int bufs, const LinearSegments sg) {
     typedef __nv_bfloat16 T;
     constexpr int NT = C * 2, W = C / 16;
     extern __shared__ __align__(16) unsigned char linear_smem[];
@@ -98,7 +106,8 @@ __global__ void __launch_bounds__(C * 2, 1) linear_chunk_kernel(const LinearArgs
                   *sb = vw + 3 * C * kLcRow;
     float *pw = reinterpret_cast<float *>(sb + 3 * (size_t)dimK * kLcRow);  // decay^0 .. decay^C
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
-    const int v0 = blockIdx.x * kLtCols, h = blockIdx.y, seq = blockIdx.z;
+    const int v0 = blockIdx.x * kLtCols, h = blockIdx.y, seg = sg.count > 1 ? blockIdx.z : 0, seq = sg.count > 1 ? 0 : blockIdx.z;
+    const int t_begin = seg * sg.tokens, t_end = sg.count > 1 ? min(a.T, t_begin + sg.tokens) : a.T;
     for (int i = tid; i <= C; i += NT) pw[i] = a.pows[(size_t)h * (kLinearPow + 1) + i];
     const int nq = s.dimP / 8, nvc = min(kLtCols, s.vP - v0) / 8;
     for (int i = tid; i < 2 * bufs * C * (dimK / 8); i += NT)  // padding columns once
@@ -112,16 +121,17 @@ __global__ void __launch_bounds__(C * 2, 1) linear_chunk_kernel(const LinearArgs
         for (int i = tid; i < C * (2 * nq + nvc); i += NT) {
             const int r = i / (2 * nq + nvc), c = i % (2 * nq + nvc);
             const T *row = y + (size_t)min(c0 + r, a.T - 1) * a.ldy;
+            if (c < nq && sg.local) continue;
             if (c < nq) cp_async16(qb + (size_t)(buf * C + r) * rs + c * 16, row + s.q_off + h * s.dimP + c * 8);
             else if (c < 2 * nq) cp_async16(kb + (size_t)(buf * C + r) * rs + (c - nq) * 16, row + s.k_off + h * s.dimP + (c - nq) * 8);
             else cp_async16(vb + (size_t)(buf * C + r) * kLcRow + (c - 2 * nq) * 16, row + s.v_off + h * s.vP + v0 + (c - 2 * nq) * 8);
         }
         cp_async_commit();
     };
-    load(0, 0);
+    load(0, t_begin);
     const int slot = a.slot_map ? a.slot_map[seq] : seq;
     float *state = a.state + ((size_t)slot * s.heads + h) * s.dim * s.vdim + v0;
-    const bool fresh = a.pos_dev[slot] == 0;
+    const bool fresh = a.pos_dev[slot] == 0 || sg.local;
     float S[MW][4][4];  // rows 16 mt + g (+ 8), columns 8 n + 2 t (+ 1); mt = warp + W * i
 #pragma unroll
     for (int i = 0; i < MW; i++)
@@ -132,15 +142,32 @@ __global__ void __launch_bounds__(C * 2, 1) linear_chunk_kernel(const LinearArgs
                 const int d = 16 * (warp + W * i) + g + 8 * (e >> 1), c = 8 * n + 2 * t + (e & 1);
                 S[i][n][e] = (!fresh && d < s.dim && v0 + c < s.vdim) ? state[(size_t)d * s.vdim + c] : 0.0f;
             }
+    if (!sg.local && seg > 0) {
+        const float d1 = a.pows[(size_t)h * (kLinearPow + 1) + kLinearPow];
+        float dl = 1.0f;
+        for (int i = 0; i < sg.tokens; i += kLinearPow) dl *= d1;
+        for (int r = 0; r < seg; r++) {
+            const float *sum = sg.sums + ((size_t)r * s.heads + h) * s.dim * s.vdim + v0;
+#pragma unroll
+            for (int i = 0; i < MW; i++)
+#pragma unroll
+                for (int n = 0; n < 4; n++)
+#pragma unroll
+                    for (int e = 0; e < 4; e++) {
+                        const int d = 16 * (warp + W * i) + g + 8 * (e >> 1), c = 8 * n + 2 * t + (e & 1);
+                        if (d < s.dim && v0 + c < s.vdim) S[i][n][e] = fmaf(S[i][n][e], dl, sum[(size_t)d * s.vdim + c]);
+                    }
+        }
+    }
     const unsigned base = (unsigned)__cvta_generic_to_shared(linear_smem);
     const unsigned qa0 = base + (warp * 16 + (lane & 15)) * rs + (lane >> 4) * 16;
     const unsigned ka0 = base + (unsigned)(kb - linear_smem) + ((lane & 7) + 8 * (lane >> 4)) * rs + ((lane >> 3) & 1) * 16;
     const unsigned kt0 = base + (unsigned)(kb - linear_smem) + ((lane >> 4) * 8 + (lane & 7)) * rs + ((lane >> 3) & 1) * 16;
     const unsigned vrow = (lane & 15) * kLcRow + (lane >> 4) * 16;
     const unsigned va0 = base + (unsigned)(vb - linear_smem) + vrow, wa0 = base + (unsigned)(vw - linear_smem) + vrow, sa0 = base + (unsigned)(sb - linear_smem) + vrow;
-    const int nchunks = (a.T + C - 1) / C;
+    const int nchunks = (t_end - t_begin + C - 1) / C;
     for (int ci = 0; ci < nchunks; ci++) {
-        const int buf = bufs == 2 ? ci & 1 : 0, c0 = ci * C, n = min(C, a.T - c0);
+        const int buf = bufs == 2 ? ci & 1 : 0, c0 = t_begin + ci * C, n = min(C, t_end - c0);
         if (bufs == 2 && ci + 1 < nchunks) {
             load(buf ^ 1, c0 + C);
             cp_async_wait<1>();
@@ -151,7 +178,7 @@ __global__ void __launch_bounds__(C * 2, 1) linear_chunk_kernel(const LinearArgs
 #pragma unroll
         for (int i = 0; i < MW; i++) {
             const int mt = warp + W * i;
-            if (mt * 16 < dimK)
+            if (mt * 16 < dimK && !sg.local)
 #pragma unroll
                 for (int nb = 0; nb < 4; nb++)
 #pragma unroll
@@ -175,7 +202,7 @@ __global__ void __launch_bounds__(C * 2, 1) linear_chunk_kernel(const LinearArgs
         }
         __syncthreads();
         const unsigned qa = qa0 + buf * C * rs, ka = ka0 + buf * C * rs, kt = kt0 + buf * C * rs, va = va0 + buf * C * kLcRow;
-        if (warp * 16 < n) {
+        if (warp * 16 < n && !sg.local) {
             float o[4][4];
 #pragma unroll
             for (int nb = 0; nb < 4; nb++) o[nb][0] = o[nb][1] = o[nb][2] = o[nb][3] = 0.0f;
@@ -271,7 +298,8 @@ __global__ void __launch_bounds__(C * 2, 1) linear_chunk_kernel(const LinearArgs
         __syncthreads();
         if (bufs == 1 && ci + 1 < nchunks) load(0, c0 + C);
     }
-    if (!a.keep_state)
+    float *out_state = sg.local ? sg.sums + ((size_t)seg * s.heads + h) * s.dim * s.vdim + v0 : state;
+    if (sg.local || (!a.keep_state && seg == sg.count - 1))
 #pragma unroll
         for (int i = 0; i < MW; i++)
 #pragma unroll
@@ -279,7 +307,7 @@ __global__ void __launch_bounds__(C * 2, 1) linear_chunk_kernel(const LinearArgs
 #pragma unroll
                 for (int e = 0; e < 4; e++) {
                     const int d = 16 * (warp + W * i) + g + 8 * (e >> 1), c = 8 * nb + 2 * t + (e & 1);
-                    if (d < s.dim && v0 + c < s.vdim) state[(size_t)d * s.vdim + c] = S[i][nb][e];
+                    if (d < s.dim && v0 + c < s.vdim) out_state[(size_t)d * s.vdim + c] = S[i][nb][e];
                 }
 }
 
@@ -319,10 +347,19 @@ int step_any(const LinearArgs &a, cudaStream_t st) {
     return fail(IM_ERR_INVALID, "linear attention is built for key dimensions up to 512 (got %d)", a.s.dim);
 }
 template <int C, int MW>
-int chunk_launch(const LinearArgs &a, int dimK, int bufs, cudaStream_t st) {
-    IM_CUDA_CHECK(launch_k(linear_chunk_kernel<C, MW>, dim3((a.s.vdim + kLtCols - 1) / kLtCols, a.s.heads, a.nseq), dim3(C * 2), linear_chunk_smem(C, dimK, bufs), st, a,
-                           dimK, bufs));
+int chunk_launch(const LinearArgs &a, int dimK, int bufs, LinearSegments sg, cudaStream_t st) {
+    const int vb = (a.s.vdim + kLtCols - 1) / kLtCols;
+    if (sg.count > 1) {
+        sg.local = 1;
+        IM_CUDA_CHECK(launch_k(linear_chunk_kernel<C, MW>, dim3(vb, a.s.heads, sg.count - 1), dim3(C * 2), linear_chunk_smem(C, dimK, bufs), st, a, dimK, bufs, sg));
+        sg.local = 0;
+    }
+    IM_CUDA_CHECK(launch_k(linear_chunk_kernel<C, MW>, dim3(vb, a.s.heads, sg.count > 1 ? sg.count : a.nseq), dim3(C * 2), linear_chunk_smem(C, dimK, bufs), st, a, dimK,
+                           bufs, sg));
     return IM_OK;
+}
+int chunk_any(const LinearArgs &a, int dimK, int bufs, const LinearSegments &sg, cudaStream_t st) {
+    return dimK <= 64 ? chunk_launch<64, 1>(a, dimK, bufs, sg, st) : dimK <= 128 ? chunk_launch<64, 2>(a, dimK, bufs, sg, st) : chunk_launch<64, 4>(a, dimK, bufs, sg, st);
 }
 
 }  // namespace
@@ -333,25 +370,34 @@ int linear_prepare(const Device *dev) {
 #define IM_SMEM(k) IM_CUDA_CHECK(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kLinearSmemMax))
     IM_SMEM((linear_step_kernel<float, 64>)); IM_SMEM((linear_step_kernel<float, 32>));
     IM_SMEM((linear_step_kernel<__nv_bfloat16, 64>)); IM_SMEM((linear_step_kernel<__nv_bfloat16, 32>));
-    IM_SMEM((linear_chunk_kernel<128, 1>)); IM_SMEM((linear_chunk_kernel<128, 2>)); IM_SMEM((linear_chunk_kernel<64, 1>)); IM_SMEM((linear_chunk_kernel<64, 2>));
+    IM_SMEM((linear_chunk_kernel<128, 1>)); IM_SMEM((linear_chunk_kernel<64, 1>)); IM_SMEM((linear_chunk_kernel<64, 2>));
     IM_SMEM((linear_chunk_kernel<64, 4>));
 #undef IM_SMEM
     return IM_OK;
 }
 
 int linear_attention_run(const Device *dev, const LinearArgs &a, cudaStream_t st, int *launches) {
-    (void)dev;
     const int dimK = round_up(a.s.dimP, 16), M = a.nseq * a.T;
     int rc = IM_ERR_BOUNDS;
-    if (!a.f32 && a.T >= 16 && dimK <= 256) {
-        if (a.T > 64) {
-            for (int bufs = 2; bufs >= 1 && rc == IM_ERR_BOUNDS; bufs--)
-                if (linear_chunk_smem(128, dimK, bufs) <= kLinearSmemMax) rc = dimK <= 128 ? chunk_launch<128, 1>(a, dimK, bufs, st) : chunk_launch<128, 2>(a, dimK, bufs, st);
+    if (!a.f32 && a.T >= 16 && dimK <= 256 && linear_chunk_smem(64, dimK, 1) <= kLinearSmemMax) {
+        LinearSegments sg;
+        sg.sums = a.seg_sums;
+        const int ctas = (a.s.vdim + kLtCols - 1) / kLtCols * a.s.heads, per_sm = 2 * linear_chunk_smem(64, dimK, 1) <= kLinearSmemMax ? 2 : 1;
+        if (a.nseq == 1 && a.T >= 2 * kLinearPow && a.seg_sums) {  // enough segments to fill the GPU
+            const int want = std::min(std::min(per_sm * dev->sm_count / ctas, a.T / kLinearPow), kLinearSegMax);
+            if (want > 1) {
+                sg.tokens = round_up((a.T + want - 1) / want, kLinearPow);
+                sg.count = (a.T + sg.tokens - 1) / sg.tokens;
+            }
         }
-        if (rc == IM_ERR_BOUNDS)
-            for (int bufs = 2; bufs >= 1 && rc == IM_ERR_BOUNDS; bufs--)
-                if (linear_chunk_smem(64, dimK, bufs) <= kLinearSmemMax)
-                    rc = dimK <= 64 ? chunk_launch<64, 1>(a, dimK, bufs, st) : dimK <= 128 ? chunk_launch<64, 2>(a, dimK, bufs, st) : chunk_launch<64, 4>(a, dimK, bufs, st);
+        if (sg.count > 1) {
+            *launches += 1;
+            rc = chunk_any(a, dimK, 1, sg, st);
+        } else if (a.T > 64 && dimK <= 128 && linear_chunk_smem(128, dimK, 2) <= kLinearSmemMax) {
+            rc = chunk_launch<128, 1>(a, dimK, 2, sg, st);
+        } else {
+            rc = chunk_any(a, dimK, linear_chunk_smem(64, dimK, 2) <= kLinearSmemMax ? 2 : 1, sg, st);
+        }
     }
     if (rc == IM_ERR_BOUNDS) rc = a.f32 ? step_any<float>(a, st) : step_any<__nv_bfloat16>(a, st);
     if (rc != IM_OK) return rc;

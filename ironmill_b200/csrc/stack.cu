@@ -70,7 +70,7 @@ struct StackModel : im_model {
     int f32 = 0, W = 0;
     DenseWeight embed, head, loop_in;
     float *embed_norm = nullptr, *final_norm = nullptr, *loop_step = nullptr;
-    float *x = nullptr, *x_alt = nullptr, *x0 = nullptr, *rec_o = nullptr, *part = nullptr, *logits = nullptr, *rows = nullptr, *hidden = nullptr;
+    float *x = nullptr, *x_alt = nullptr, *x0 = nullptr, *rec_o = nullptr, *seg_sums = nullptr, *part = nullptr, *logits = nullptr, *rows = nullptr, *hidden = nullptr;
     void *y = nullptr, *cat = nullptr, *h = nullptr, *qabs = nullptr, *kv = nullptr;
     int ldy = 0, ldcat = 0;
     size_t part_bytes = 0, kv_bytes = 0;
@@ -325,7 +325,7 @@ int StackModel::finalize() {
     }
     if (has_latent && wide) cfg.prefill_chunk_size = std::min(cfg.prefill_chunk_size, kStackChunkWide);
     MT = std::max(std::max(cfg.max_batch, cfg.prefill_chunk_size), std::min(kAllLogitsChunk, cfg.max_seq_len));
-    size_t abs_elems = 0, rec_elems = 0, kv_need = 0;
+    size_t abs_elems = 0, rec_elems = 0, seg_elems = 0, kv_need = 0;
     for (StackLayer &L : layers) {
         ldy = std::max(ldy, L.pair0);
         ldcat = std::max(ldcat, L.mixP + L.ffP);
@@ -339,6 +339,7 @@ int StackModel::finalize() {
             if (!wide) kv_need = std::max(kv_need, std::max(head_bytes, std::min(kExpandBytes, head_bytes * L.ls.heads)));
         } else {
             rec_elems = std::max(rec_elems, (size_t)MT * L.ns.heads * L.ns.vP);
+            if (!f32 && MT >= 2 * kLinearPow) seg_elems = std::max(seg_elems, (size_t)(kLinearSegMax - 1) * L.ns.heads * L.ns.dim * L.ns.vdim);
         }
     }
     ldy = std::max(ldy, 8);
@@ -359,6 +360,7 @@ int StackModel::finalize() {
     IM_TRY(alloc(&kv, kv_need));
     kv_bytes = kv_need;
     IM_TRY(alloc((void **)&rec_o, rec_elems * 4));
+    IM_TRY(alloc((void **)&seg_sums, seg_elems * 4));
     if (rec_elems) IM_CUDA_CHECK(cudaMemset(rec_o, 0, rec_elems * 4));
     IM_TRY(alloc((void **)&logits, slots * cfg.vocab_size * 4));
     logits_dev = logits;
@@ -418,7 +420,7 @@ int StackModel::forward(int nseq, int T, cudaStream_t st, int *launches, Prof *p
         } else {
             LinearArgs a{};
             a.s = L.ns; a.f32 = f32; a.y = y; a.ldy = ldy; a.norm = L.o_norm; a.pows = L.pows; a.state = static_cast<float *>(r.cache);
-            a.nseq = nseq; a.T = T; a.pos_dev = pos_dev; a.slot_map = slots; a.keep_state = uncounted ? 1 : 0; a.o = rec_o; a.out = cat; a.ldo = ldcat;
+            a.nseq = nseq; a.T = T; a.pos_dev = pos_dev; a.slot_map = slots; a.keep_state = uncounted ? 1 : 0; a.o = rec_o; a.seg_sums = seg_sums; a.out = cat; a.ldo = ldcat;
             IM_TRY(linear_attention_run(dev, a, st, &nl));
         }
         IM_MARK(kCatAttn);

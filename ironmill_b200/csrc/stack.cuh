@@ -123,10 +123,12 @@ struct LinearArgs {
     const int *pos_dev, *slot_map;
     int keep_state;     // 1: leave the state as it was (a pass that is not counted)
     float *o;           // [M, heads * vP] f32 scratch
+    float *seg_sums;    // [kLinearSegMax - 1][heads][dim][vdim] f32 scratch of a long prompt's segments (optional)
     void *out;          // [M, ldo]
     int ldo;
 };
 constexpr int kLinearPow = 128;
+constexpr int kLinearSegMax = 8;
 int linear_attention_run(const Device *dev, const LinearArgs &a, cudaStream_t st, int *launches);
 int linear_prepare(const Device *dev);
 
