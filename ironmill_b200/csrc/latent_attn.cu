@@ -213,9 +213,11 @@ __global__ void __launch_bounds__(kLaWarps * 32, 1) latent_attn_kernel(const Lat
     const __nv_bfloat16 *cache = static_cast<const __nv_bfloat16 *>(a.cache) + (size_t)slot * a.max_seq * s.rowP;
     auto load_tile = [&](int buf, int p0) {
         unsigned char *dst = kt + (size_t)buf * kLaN * rs;
-        for (int i = tid; i < kLaN * nch; i += NT) {
-            const int r = i / nch, c = i % nch;
-            cp_async16(dst + r * rs + c * 16, cache + (size_t)min(p0 + r, r1 - 1) * s.rowP + c * 8);
+#pragma unroll
+        for (int j = 0; j < kLaN / kLaWarps; j++) {  // a warp per cached row
+            const int r = warp + j * kLaWarps;
+            const __nv_bfloat16 *src = cache + (size_t)min(p0 + r, r1 - 1) * s.rowP;
+            for (int c = lane; c < nch; c += 32) cp_async16(dst + r * rs + c * 16, src + c * 8);
         }
         cp_async_commit();
     };
@@ -457,45 +459,48 @@ __device__ __forceinline__ float row_norm(const LatentPart &p, size_t row, float
     return 1.0f / l;
 }
 
-// grid (rows, column blocks of 128): the splits of a row added up and normalised
-__global__ void __launch_bounds__(128) latent_combine_kernel(const LatentPart p, const float *__restrict__ sink, int heads, int latP, float *__restrict__ out) {
-    __shared__ float wk[256], sm[4], sl[4];
+// grid (rows, column blocks of 128), 512 threads: the splits of a row added up (a quarter of them per group of 128 threads)
+// and normalised
+constexpr int kLcThreads = 512;
+__global__ void __launch_bounds__(kLcThreads) latent_combine_kernel(const LatentPart p, const float *__restrict__ sink, int heads, int latP, float *__restrict__ out) {
+    __shared__ float wk[256], sm[8], sl[8], part[3][128];
     const size_t row = blockIdx.x;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const float s = sink ? sink[row % heads] : -INFINITY;
     pdl_trigger();
     pdl_wait();
-    float m[2], l[2];
-#pragma unroll
-    for (int i = 0; i < 2; i++) {
-        const int k = tid + 128 * i;
-        m[i] = k < p.splits ? p.pm[row * p.splits + k] : -INFINITY;
-        l[i] = k < p.splits ? p.pl[row * p.splits + k] : 0.0f;
+    float m = -INFINITY, l = 0.0f;
+    if (tid < p.splits) {
+        m = p.pm[row * p.splits + tid];
+        l = p.pl[row * p.splits + tid];
     }
-    float gm = warp_max(fmaxf(m[0], m[1]));
-    if (lane == 0) sm[warp] = gm;
+    const float wm = warp_max(m);
+    if (lane == 0 && warp < 8) sm[warp] = wm;
     __syncthreads();
-    gm = fmaxf(fmaxf(fmaxf(sm[0], sm[1]), fmaxf(sm[2], sm[3])), s);
-    float sum = 0.0f;
+    float gm = s;
 #pragma unroll
-    for (int i = 0; i < 2; i++) {
-        m[i] = m[i] == -INFINITY ? 0.0f : expf(m[i] - gm);
-        wk[tid + 128 * i] = m[i];
-        sum = fmaf(l[i], m[i], sum);
-    }
-    sum = warp_sum(sum);
-    if (lane == 0) sl[warp] = sum;
+    for (int i = 0; i < 8; i++) gm = fmaxf(gm, sm[i]);
+    const float w = m == -INFINITY ? 0.0f : expf(m - gm), ws = warp_sum(l * w);
+    if (tid < 256) wk[tid] = w;
+    if (lane == 0 && warp < 8) sl[warp] = ws;
     __syncthreads();
-    const float inv = 1.0f / (sl[0] + sl[1] + sl[2] + sl[3] + (s == -INFINITY ? 0.0f : expf(s - gm)));
-    const int c = blockIdx.y * 128 + tid;
-    if (c >= latP) return;
+    float sum = s == -INFINITY ? 0.0f : expf(s - gm);
+#pragma unroll
+    for (int i = 0; i < 8; i++) sum += sl[i];
+    const int grp = tid >> 7, c = blockIdx.y * 128 + (tid & 127);
+    const int per = (p.splits + 3) / 4, k0 = grp * per, k1 = min(p.splits, k0 + per);
     float acc = 0.0f;
+    if (c < latP) {
+        const float *src = p.po + row * p.splits * latP + c;
 #pragma unroll 8
-    for (int k = 0; k < p.splits; k++) {
-        const float w = wk[k];
-        if (w != 0.0f) acc = fmaf(w, p.po[(row * p.splits + k) * latP + c], acc);
+        for (int k = k0; k < k1; k++) {
+            const float v = src[(size_t)k * latP], wt = wk[k];  // a split without positions left its sums unwritten
+            acc += wt == 0.0f ? 0.0f : wt * v;
+        }
     }
-    out[row * latP + c] = acc * inv;
+    if (grp) part[grp - 1][tid & 127] = acc;
+    __syncthreads();
+    if (grp == 0 && c < latP) out[row * latP + c] = (acc + part[0][tid] + part[1][tid] + part[2][tid]) / sum;
 }
 
 // grid (heads, slices of the value rows, token groups of MB): out[m, h] = W_uv[h] o'.  src: the normalised sums, or (single
@@ -577,12 +582,15 @@ __global__ void __launch_bounds__(kLpThreads, DV <= 128 ? 3 : 1) latent_prefill_
     auto load_tile = [&](int buf, int p0) {
         const __nv_bfloat16 *kvh = kv + (size_t)hl * (s.dimP + s.vP);
         unsigned char *kd = kt + (size_t)buf * kLpN * rs, *vd = vt + (size_t)buf * kLpN * vs;
-        for (int i = tid; i < kLpN * (nk + nr + nvv); i += NT) {
-            const int r = i / (nk + nr + nvv), c = i % (nk + nr + nvv);
+        // the chunks of a row: [key | value] as they lie in kv, then the rotated part from the cache
+        for (int r = warp; r < kLpN; r += kLpThreads / 32) {
             const size_t p = (size_t)min(p0 + r, n_end - 1);
-            if (c < nk) cp_async16(kd + r * rs + c * 16, kvh + p * ldkv + c * 8);
-            else if (c < nk + nr) cp_async16(kd + r * rs + c * 16, cache + p * s.rowP + s.latP + (c - nk) * 8);
-            else cp_async16(vd + r * vs + (c - nk - nr) * 16, kvh + p * ldkv + s.dimP + (c - nk - nr) * 8);
+            const __nv_bfloat16 *krow = kvh + p * ldkv, *rrow = cache + p * s.rowP + s.latP;
+            for (int c = lane; c < nk + nvv + nr; c += 32) {
+                const bool key = c < nk, rot = c >= nk + nvv;
+                unsigned char *dst = key ? kd + r * rs + c * 16 : rot ? kd + r * rs + (c - nvv) * 16 : vd + r * vs + (c - nk) * 16;
+                cp_async16(dst, rot ? rrow + (c - nk - nvv) * 8 : krow + c * 8);
+            }
         }
         cp_async_commit();
     };
@@ -590,6 +598,9 @@ __global__ void __launch_bounds__(kLpThreads, DV <= 128 ? 3 : 1) latent_prefill_
     const int tok0 = tb * kLpM + warp * 16 + g, tok1 = tok0 + 8;
     const int lim[2] = {tok0 < a.T ? P + tok0 : -1, tok1 < a.T ? P + tok1 : -1};
     const int warp_end = P + min(tb * kLpM + warp * 16 + 16, a.T);  // tiles from here on are masked for the whole warp
+    const int warp_full = tb * kLpM + warp * 16 + 16 <= a.T ? P + tb * kLpM + warp * 16 : -1;  // every row sees the positions up to here
+    constexpr float kLog2e = 1.4426950408889634f;
+    const float scale2 = s.scale * kLog2e;  // scores in units of log 2: one exponential instruction each
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};
     float o[ND][4];
 #pragma unroll
@@ -624,28 +635,43 @@ __global__ void __launch_bounds__(kLpThreads, DV <= 128 ? 3 : 1) latent_prefill_
                 }
             }
             float corr[2], mx[2] = {-INFINITY, -INFINITY};
+            if (p0 + kLpN - 1 <= warp_full) {
 #pragma unroll
-            for (int nb = 0; nb < kLpNB; nb++)
+                for (int nb = 0; nb < kLpNB; nb++)
 #pragma unroll
-                for (int e = 0; e < 4; e++) {
-                    const int p = p0 + 8 * nb + 2 * t + (e & 1);
-                    sc[nb][e] = p <= lim[e >> 1] ? sc[nb][e] * s.scale : -INFINITY;
-                    mx[e >> 1] = fmaxf(mx[e >> 1], sc[nb][e]);
-                }
+                    for (int e = 0; e < 4; e++) {
+                        sc[nb][e] *= scale2;
+                        mx[e >> 1] = fmaxf(mx[e >> 1], sc[nb][e]);
+                    }
+            } else {
+#pragma unroll
+                for (int nb = 0; nb < kLpNB; nb++)
+#pragma unroll
+                    for (int e = 0; e < 4; e++) {
+                        const int p = p0 + 8 * nb + 2 * t + (e & 1);
+                        sc[nb][e] = p <= lim[e >> 1] ? sc[nb][e] * scale2 : -INFINITY;
+                        mx[e >> 1] = fmaxf(mx[e >> 1], sc[nb][e]);
+                    }
+            }
+            bool moved = false;
 #pragma unroll
             for (int r = 0; r < 2; r++) {
                 mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
                 mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
                 const float m_new = fmaxf(m_run[r], mx[r]);
-                corr[r] = m_new == -INFINITY ? 1.0f : __expf(m_run[r] - m_new);
+                moved |= m_new > m_run[r];
+                corr[r] = m_new == -INFINITY ? 1.0f : exp2f(m_run[r] - m_new);
                 m_run[r] = m_new;
                 l_run[r] *= corr[r];
             }
+            if (__any_sync(0xffffffffu, moved)) {
 #pragma unroll
-            for (int i = 0; i < ND; i++) {
-                o[i][0] *= corr[0]; o[i][1] *= corr[0];
-                o[i][2] *= corr[1]; o[i][3] *= corr[1];
+                for (int i = 0; i < ND; i++) {
+                    o[i][0] *= corr[0]; o[i][1] *= corr[0];
+                    o[i][2] *= corr[1]; o[i][3] *= corr[1];
+                }
             }
+            const float base[2] = {m_run[0] == -INFINITY ? 0.0f : m_run[0], m_run[1] == -INFINITY ? 0.0f : m_run[1]};
 #pragma unroll
             for (int kb = 0; kb < kLpN / 16; kb++) {
                 unsigned hi[4], lo[4];
@@ -654,7 +680,7 @@ __global__ void __launch_bounds__(kLpThreads, DV <= 128 ? 3 : 1) latent_prefill_
 #pragma unroll
                     for (int r = 0; r < 2; r++) {
                         const float s0 = sc[2 * kb + hb][2 * r], s1 = sc[2 * kb + hb][2 * r + 1];
-                        const float w0 = s0 == -INFINITY ? 0.0f : __expf(s0 - m_run[r]), w1 = s1 == -INFINITY ? 0.0f : __expf(s1 - m_run[r]);
+                        const float w0 = exp2f(s0 - base[r]), w1 = exp2f(s1 - base[r]);  // a masked score gives zero
                         l_run[r] += w0 + w1;
                         unsigned terms[2];
                         split_bf2<2>(w0, w1, terms);
@@ -674,7 +700,7 @@ __global__ void __launch_bounds__(kLpThreads, DV <= 128 ? 3 : 1) latent_prefill_
         }
         __syncthreads();
     }
-    const float sink = a.sink ? a.sink[h] : -INFINITY;
+    const float sink = a.sink ? a.sink[h] * kLog2e : -INFINITY;
 #pragma unroll
     for (int r = 0; r < 2; r++) {
         float l = l_run[r];
@@ -682,8 +708,8 @@ __global__ void __launch_bounds__(kLpThreads, DV <= 128 ? 3 : 1) latent_prefill_
         l += __shfl_xor_sync(0xffffffffu, l, 2);
         const int tok = r == 0 ? tok0 : tok1;
         if (tok < a.T) {
-            const float gm = fmaxf(m_run[r], sink), c = __expf(m_run[r] - gm);
-            const float inv = c / (l * c + (sink == -INFINITY ? 0.0f : __expf(sink - gm)));
+            const float gm = fmaxf(m_run[r], sink), c = exp2f(m_run[r] - gm);
+            const float inv = c / (l * c + (sink == -INFINITY ? 0.0f : exp2f(sink - gm)));
             __nv_bfloat16 *dst = static_cast<__nv_bfloat16 *>(a.out) + (size_t)tok * a.ldo + h * s.vP;
 #pragma unroll
             for (int nd = 0; nd < ND; nd++) {
@@ -841,7 +867,7 @@ int latent_attention_run(const Device *dev, const LatentArgs &a, cudaStream_t st
     }
     const float *src = p.po;
     if (splits > 1) {
-        IM_CUDA_CHECK(launch_k(latent_combine_kernel, dim3((unsigned)rows, (s.latP + 127) / 128), dim3(128), 0, st, p, a.sink, s.heads, s.latP, comb));
+        IM_CUDA_CHECK(launch_k(latent_combine_kernel, dim3((unsigned)rows, (s.latP + 127) / 128), dim3(kLcThreads), 0, st, p, a.sink, s.heads, s.latP, comb));
         src = comb;
         *launches += 1;
     }

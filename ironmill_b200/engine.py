@@ -263,6 +263,20 @@ class CudaInference:
         self._next = nxt
         return [(int(sid), out[i]) for i, sid in enumerate(ids)]
 
+    def generate(self, prompts, max_new_tokens: int) -> list:
+        """Greedy continuations of several prompts, decoded together as sequences of one batch (add_sequence,
+        batch_decode_step); one list of token ids per prompt."""
+        ids = [self.add_sequence(p) for p in prompts]
+        out = {i: [] for i in ids}
+        for n in range(max_new_tokens):
+            for i in ids:
+                out[i].append(self._next[i])
+            if n + 1 < max_new_tokens:
+                self.batch_decode_step({i: self._next[i] for i in ids})
+        for i in ids:
+            self.remove_sequence(i)
+        return [out[i] for i in ids]
+
     @_wrap
     def test_missing_ranks(self, n: int) -> None:
         """Host-side fault injection (tests of the error path; `decode_schedule="tagged"` on one GPU only): n = 1 makes

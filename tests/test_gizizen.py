@@ -139,3 +139,34 @@ def test_a_lost_state_or_key_shows():
             if what == "lat" and "lat" in st:
                 st["lat"] = [r * (i != 31) for i, r in enumerate(st["lat"])]
         assert G.error(m.forward(toks[60:]), right) > G.TOL["bfloat16"]
+
+
+def test_trace_replay_drives_the_sequence_interface(tmp_path):
+    """Portions, wanted places in any order, slots given back; the engine is a stand-in that records calls."""
+    from ironmill_b200.trace import replay
+
+    class Engine:
+        def __init__(self):
+            self.live, self.calls = set(), []
+
+        def open_sequence(self):
+            i = min(set(range(9)) - self.live)
+            self.live.add(i)
+            return i
+
+        def extend_sequence(self, sid, tokens, want):
+            self.calls.append((sid, list(tokens), list(want)))
+            return np.array([[sid, tokens[k], 0.5] for k in want], dtype=np.float32).reshape(len(want), 3)
+
+        def remove_sequence(self, sid):
+            self.live.remove(sid)
+
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": [4, 5, 6], "want": [2, 0]}], "end": []},
+             {"step": 1, "entries": [{"id": "b", "tokens": [7], "want": []}, {"id": "a", "tokens": [8], "want": []}], "end": ["a"]},
+             {"step": 2, "entries": [{"id": "c", "tokens": [9, 1], "want": [1]}], "end": ["b", "c"]}]
+    e, said = Engine(), []
+    replay(e, [json.dumps(s) + "\n" for s in steps], str(tmp_path), said.append)
+    assert said == ["done 0", "done 1", "done 2"] and not e.live
+    assert e.calls == [(0, [4, 5, 6], [0, 2]), (1, [7], []), (0, [8], []), (0, [9, 1], [1])]
+    assert np.fromfile(tmp_path / "0.f32", "<f4").reshape(-1, 3)[:, 1].tolist() == [6, 4]
+    assert not (tmp_path / "1.f32").exists() and np.fromfile(tmp_path / "2.f32", "<f4").tolist() == [0, 1, 0.5]

@@ -3,6 +3,7 @@ portions, token by token, in batches and slots, through the engine's own entry p
 import json
 import os
 import subprocess
+import sys
 
 import numpy as np
 import pytest
@@ -141,6 +142,21 @@ def test_a_far_key_at_every_border(dtype, wide):
         assert G.error(e.decode_step(int(toks[-1]))[None], want) < G.TOL[dtype]
 
 
+def test_prompts_long_enough_for_parallel_segments():
+    """bf16: a 900-token prompt's recurrence runs in segments; cut elsewhere it does not; then decoding from the state."""
+    cfg = G.config([G.lightning(heads=2, dim=36, vdim=40, decay=(0.995, 0.9999)), G.lightning(heads=1, dim=72, vdim=20, decay=(0.98,), ff=0)])
+    w = G.weights(cfg, 30)
+    toks = tokens(920, 203)
+    want = OracleGizizen(cfg, w).forward(toks)
+    e = engine(cfg, w, "bfloat16", max_seq_len=920)
+    for first in (0, 37, 300):
+        e.reset()
+        if first:
+            e.prefill(toks[:first])
+        assert G.error(e.prefill(toks[first:900])[None], want[899:900]) < G.TOL["bfloat16"]
+        assert G.error(decoded(e, toks[900:]), want[900:]) < G.TOL["bfloat16"]
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_first_tokens(dtype):
     """Sequences of one token and a few, in one portion and one by one."""
@@ -233,6 +249,26 @@ def test_greedy_generation():
         for sid, logits in e.batch_decode_step():
             seen[sid].append(int(np.argmax(logits)))
     assert seen[ids[0]] == seen[ids[2]] == picks[:11] and seen[ids[1]] != picks[:11]
+    e.reset()
+    rows = e.generate([prompt, prompt[:20]], 12)
+    assert rows[0] == picks[:12] and rows[1] == seen[ids[1]] + rows[1][11:]
+
+
+def test_command_line_generation(tmp_path):
+    """The same continuation from a checkpoint folder and from a bundle written from it."""
+    from ironmill_b200.bundle import write_gpu_bundle
+    w = G.weights(MIX, 21)
+    prompt = tokens(40, 203)
+    e = engine(MIX, w, "float32", max_seq_len=128)
+    want = e.generate([prompt], 8)[0]
+    G.write_checkpoint(tmp_path / "model", MIX, w)
+    p = G.Provider(MIX, w)
+    write_gpu_bundle(str(tmp_path / "bundle"), p.config(), {n: p.tensor(n) for n in p.tensor_names()})
+    for folder in ("model", "bundle"):
+        r = subprocess.run([sys.executable, "-m", "ironmill_b200", "generate", "--model", str(tmp_path / folder), "--dtype", "float32", "--max-new-tokens", "8",
+                            "--tokens", ",".join(map(str, prompt))], capture_output=True, text=True, timeout=200, cwd=ROOT)
+        assert r.returncode == 0, r.stderr[-2000:]
+        assert [int(t) for t in r.stdout.split(",")] == want
 
 
 def test_repeated_steps_are_bit_identical():
