@@ -459,11 +459,12 @@ __device__ __forceinline__ float row_norm(const LatentPart &p, size_t row, float
     return 1.0f / l;
 }
 
-// grid (rows, column blocks of 128), 512 threads: the splits of a row added up (a quarter of them per group of 128 threads)
-// and normalised
-constexpr int kLcThreads = 512;
-__global__ void __launch_bounds__(kLcThreads) latent_combine_kernel(const LatentPart p, const float *__restrict__ sink, int heads, int latP, float *__restrict__ out) {
-    __shared__ float wk[256], sm[8], sl[8], part[3][128];
+// grid (rows, column blocks of 128), GR groups of 128 threads: the splits of a row (at most 256, or 128 for one group) added
+// up, a share of them per group, and normalised
+template <int GR>
+__global__ void __launch_bounds__(GR * 128) latent_combine_kernel(const LatentPart p, const float *__restrict__ sink, int heads, int latP, float *__restrict__ out) {
+    constexpr int NW = GR == 1 ? 4 : 8;  // warps that hold a split's maximum
+    __shared__ float wk[NW * 32], sm[NW], sl[NW], part[GR][128];
     const size_t row = blockIdx.x;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const float s = sink ? sink[row % heads] : -INFINITY;
@@ -475,20 +476,20 @@ __global__ void __launch_bounds__(kLcThreads) latent_combine_kernel(const Latent
         l = p.pl[row * p.splits + tid];
     }
     const float wm = warp_max(m);
-    if (lane == 0 && warp < 8) sm[warp] = wm;
+    if (lane == 0 && warp < NW) sm[warp] = wm;
     __syncthreads();
     float gm = s;
 #pragma unroll
-    for (int i = 0; i < 8; i++) gm = fmaxf(gm, sm[i]);
+    for (int i = 0; i < NW; i++) gm = fmaxf(gm, sm[i]);
     const float w = m == -INFINITY ? 0.0f : expf(m - gm), ws = warp_sum(l * w);
-    if (tid < 256) wk[tid] = w;
-    if (lane == 0 && warp < 8) sl[warp] = ws;
+    if (warp < NW) wk[tid] = w;
+    if (lane == 0 && warp < NW) sl[warp] = ws;
     __syncthreads();
     float sum = s == -INFINITY ? 0.0f : expf(s - gm);
 #pragma unroll
-    for (int i = 0; i < 8; i++) sum += sl[i];
+    for (int i = 0; i < NW; i++) sum += sl[i];
     const int grp = tid >> 7, c = blockIdx.y * 128 + (tid & 127);
-    const int per = (p.splits + 3) / 4, k0 = grp * per, k1 = min(p.splits, k0 + per);
+    const int per = (p.splits + GR - 1) / GR, k0 = grp * per, k1 = min(p.splits, k0 + per);
     float acc = 0.0f;
     if (c < latP) {
         const float *src = p.po + row * p.splits * latP + c;
@@ -498,9 +499,13 @@ __global__ void __launch_bounds__(kLcThreads) latent_combine_kernel(const Latent
             acc += wt == 0.0f ? 0.0f : wt * v;
         }
     }
-    if (grp) part[grp - 1][tid & 127] = acc;
-    __syncthreads();
-    if (grp == 0 && c < latP) out[row * latP + c] = (acc + part[0][tid] + part[1][tid] + part[2][tid]) / sum;
+    if (GR > 1) {
+        part[grp][tid & 127] = acc;
+        __syncthreads();
+#pragma unroll
+        for (int i = 1; i < GR; i++) acc += part[i][tid & 127];
+    }
+    if (grp == 0 && c < latP) out[row * latP + c] = acc / sum;
 }
 
 // grid (heads, slices of the value rows, token groups of MB): out[m, h] = W_uv[h] o'.  src: the normalised sums, or (single
@@ -867,7 +872,9 @@ int latent_attention_run(const Device *dev, const LatentArgs &a, cudaStream_t st
     }
     const float *src = p.po;
     if (splits > 1) {
-        IM_CUDA_CHECK(launch_k(latent_combine_kernel, dim3((unsigned)rows, (s.latP + 127) / 128), dim3(kLcThreads), 0, st, p, a.sink, s.heads, s.latP, comb));
+        const dim3 grid((unsigned)rows, (s.latP + 127) / 128);
+        if (splits > 32) IM_CUDA_CHECK(launch_k(latent_combine_kernel<4>, grid, dim3(512), 0, st, p, a.sink, s.heads, s.latP, comb));
+        else IM_CUDA_CHECK(launch_k(latent_combine_kernel<1>, grid, dim3(128), 0, st, p, a.sink, s.heads, s.latP, comb));
         src = comb;
         *launches += 1;
     }

@@ -126,7 +126,7 @@ def test_a_far_key_at_every_border(dtype, wide):
     score = q @ (lat @ w["l0.mix.uk"][:d].T.astype(np.float64)).T * mx["scale"]
     asks, needle = np.unravel_index(np.argmax(score), score.shape)
     dull = np.argsort(score[asks])[:40]
-    e = engine(cfg, w, dtype, max_seq_len=2048)
+    e = engine(cfg, w, dtype, max_seq_len=4096)  # more splits than one group of threads adds up
     rng = np.random.default_rng(15)
     for n, at in ((200, 0), (200, 63), (200, 64), (200, 65), (200, 127), (200, 128), (200, 198), (517, 0), (517, 191), (517, 511), (517, 512), (70, 3)):
         toks = rng.choice(dull, n).astype(np.uint32)
