@@ -326,23 +326,42 @@ typedef struct im_model_config {
 int im_cuda_model_create(im_device *dev, const im_model_config *cfg, im_model **out);
 
 /* Models given as a list of layers (no counterpart in the reference, whose model types are fixed transformer blocks).
- * A layer adds mixer(n) + ffn(n) to the residual, n = rms_norm(residual) * norm1 (a parallel block); the mixer is one of the
- * kinds below and ff = 0 leaves the feed-forward out.  Layers loop_start .. loop_stop - 1 run loop_times times in a row with
+ * A layer is a mixer of one of the kinds below and a feed-forward down(act(gate h) * up h) (ff = 0 leaves it out), joined to the
+ * residual x in one of two ways:
+ *   IM_BLOCK_PARALLEL  x += mixer(n) + ffn(n), n = rms_norm(x) * norm1
+ *   IM_BLOCK_POSTNORM  x += rms_norm(mixer(x)) * norm1, then x += rms_norm(ffn(x)) * norm2
+ * Layers loop_start .. loop_stop - 1 run loop_times times in a row with
  * the same weights and a cache of their own each time; before every such pass the residual becomes
  * W_in [residual, embedding output] + step[pass].  loop_times = 0: no loop.
  * Everything after model_create_stack is the ordinary im_model: finalize, prefill, decode, sequences. */
 #define IM_MIXER_LATENT 1   /* latent attention: cached [normed latent | rotated key part], softmax with a sink logit per head */
 #define IM_MIXER_LINEAR 2   /* decayed linear attention: f32 state [dim, vdim] per head, normed and gated output */
+#define IM_MIXER_GROUPED 3  /* grouped-query attention over cached keys and values: normed, rotated queries and keys, a sink logit per
+                             * head, an output gate, optionally chunked */
+#define IM_MIXER_GATED 4    /* linear attention whose decay is a function of the token, one per key channel; output normed per head
+                             * and gated */
+#define IM_BLOCK_PARALLEL 0
+#define IM_BLOCK_POSTNORM 1
+#define IM_ACT_GELU_TANH 0
+#define IM_ACT_SILU 1
 typedef struct im_stack_layer {
     int mixer, heads, dim, vdim; /* dim: (unrotated) query / key size of a head, vdim: value size */
-    int ff;                      /* feed-forward width, gelu_tanh(gate) * up; 0 = none */
-    /* IM_MIXER_LATENT */
-    int kv_rank, rot_dim, rot_dims; /* latent size; rotated query / key size; how much of it is rotated */
+    int ff;                      /* feed-forward width; 0 = none */
+    /* IM_MIXER_LATENT, IM_MIXER_GROUPED */
+    int kv_rank, rot_dim, rot_dims; /* latent: latent size, rotated query / key size; how many dimensions are rotated */
     float scale;
     double rot_base;
     double yarn_factor, yarn_original, yarn_fast, yarn_slow; /* interpolation of long contexts; factor 0 = plain rotation */
     /* IM_MIXER_LINEAR */
     const double *decay_host;    /* [heads] */
+    /* IM_MIXER_GROUPED */
+    int kv_heads;                /* query head h reads key / value head h / (heads / kv_heads) */
+    int chunk;                   /* position i sees j <= i of its own chunk of this many positions; 0 = all j <= i */
+    int kv_from;                 /* 0: keys and values of its own; n > 0: those of layer n - 1 (an earlier grouped layer) */
+    double rot_divide;           /* every frequency is divided by this (0 = 1) */
+    /* IM_MIXER_GATED */
+    int gate_rank;               /* decay = sigmoid(a2 (a1 h) + b)^(1 / tau), a1 [gate_rank, width] */
+    float tau;
 } im_stack_layer;
 typedef struct im_stack_config {
     int vocab, width, num_layers;
@@ -350,13 +369,19 @@ typedef struct im_stack_config {
     int loop_start, loop_stop, loop_times;
     float norm_eps;
     float logit_softcap;         /* 0 = none */
+    int block;                   /* IM_BLOCK_... */
+    int ff_act;                  /* IM_ACT_... of the feed-forwards */
+    float embed_scale;           /* 0: the embedding is rms_norm(row) * embed.norm; otherwise row * embed_scale (no embed.norm) */
+    int tied_head;               /* 1: the embedding table (without its scale) is the output head */
     int max_seq_len, max_batch;  /* 0 = 2048 / 1 */
     int prefill_chunk_size;      /* 0 = the largest */
     int compute_f32;             /* 0: weights, activations and latent caches in bf16; 1: everything in f32 */
 } im_stack_config;
 int im_cuda_model_create_stack(im_device *dev, const im_stack_config *cfg, im_model **out);
 /* Tensors of such a model under their checkpoint names: embed, embed.norm, loop.in, loop.step, l<i>.norm1,
- * l<i>.mix.{q,dkv,dkv.norm,uk,uv,sink,o} or l<i>.mix.{q,k,v,g,o,norm}, l<i>.mlp.{gate,up,down}, final.norm, head.
+ * l<i>.norm2 (post-norm blocks with a feed-forward), l<i>.mix.{q,dkv,dkv.norm,uk,uv,sink,o} (latent), l<i>.mix.{q,k,v,g,o,norm} (linear),
+ * l<i>.mix.{q,q.norm,sink,g,o} and without kv_from .{k,v,k.norm} (grouped), l<i>.mix.{q,k,v,g,o,norm,a1,a2,a2.b} (gated),
+ * l<i>.mlp.{gate,up,down}, final.norm, head.
  * Row-major [out, in]; dtype IM_DTYPE_F16 / F32 / BF16; converted to the compute type (norm weights, sinks, steps: f32). */
 int im_cuda_model_load_tensor(im_model *m, const char *name, const void *data_host, int dtype, int ndim, const int64_t *shape);
 void im_cuda_model_free(im_model *m);

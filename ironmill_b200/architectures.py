@@ -10,7 +10,7 @@ import numpy as np
 
 from ._lib import IM_DTYPE_BF16, IM_DTYPE_F16, IM_DTYPE_F32, check, lib, vp
 from .bundle import GpuBundleError, ModelConfig
-from .stack_config import LatentAttention, LinearAttention, StackConfig
+from .stack_config import DESIGNS, GatedLinearAttention, GroupedAttention, LatentAttention, LinearAttention, StackConfig
 
 
 class _CModelConfig(C.Structure):
@@ -26,14 +26,15 @@ class _CModelConfig(C.Structure):
 class _CStackLayer(C.Structure):
     _fields_ = [("mixer", C.c_int), ("heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("ff", C.c_int), ("kv_rank", C.c_int),
                 ("rot_dim", C.c_int), ("rot_dims", C.c_int), ("scale", C.c_float), ("rot_base", C.c_double), ("yarn_factor", C.c_double),
-                ("yarn_original", C.c_double), ("yarn_fast", C.c_double), ("yarn_slow", C.c_double), ("decay", C.POINTER(C.c_double))]
+                ("yarn_original", C.c_double), ("yarn_fast", C.c_double), ("yarn_slow", C.c_double), ("decay", C.POINTER(C.c_double)),
+                ("kv_heads", C.c_int), ("chunk", C.c_int), ("kv_from", C.c_int), ("rot_divide", C.c_double), ("gate_rank", C.c_int), ("tau", C.c_float)]
 
 
 class _CStackConfig(C.Structure):
     _fields_ = [("vocab", C.c_int), ("width", C.c_int), ("num_layers", C.c_int), ("layers", C.POINTER(_CStackLayer)),
                 ("loop_start", C.c_int), ("loop_stop", C.c_int), ("loop_times", C.c_int), ("norm_eps", C.c_float),
-                ("logit_softcap", C.c_float), ("max_seq_len", C.c_int), ("max_batch", C.c_int), ("prefill_chunk_size", C.c_int),
-                ("compute_f32", C.c_int)]
+                ("logit_softcap", C.c_float), ("block", C.c_int), ("ff_act", C.c_int), ("embed_scale", C.c_float), ("tied_head", C.c_int),
+                ("max_seq_len", C.c_int), ("max_batch", C.c_int), ("prefill_chunk_size", C.c_int), ("compute_f32", C.c_int)]
 
 
 class QuantizedBlocks:
@@ -41,6 +42,10 @@ class QuantizedBlocks:
     native = "quantized"
     library = None           # part of the complete library only
     config = ModelConfig
+
+    @staticmethod
+    def complete(mc: ModelConfig, provider) -> None:
+        """Sizes that only the tensors give: none."""
 
     @staticmethod
     def create(engine, mc: ModelConfig) -> C.c_void_p:
@@ -99,6 +104,11 @@ class LayerStack:
     config = StackConfig
 
     @staticmethod
+    def complete(mc: StackConfig, provider) -> None:
+        """Sizes that only the tensors' shapes give."""
+        mc.complete(lambda name: tuple(provider.tensor(name).shape) if provider.has_tensor(name) else None)
+
+    @staticmethod
     def create(engine, mc: StackConfig) -> C.c_void_p:
         cfg = engine.config
         if cfg.tp_world != 1:
@@ -115,8 +125,15 @@ class LayerStack:
                 c.mixer = 2
                 keep.append((C.c_double * m.heads)(*m.decay))
                 c.decay = C.cast(keep[-1], C.POINTER(C.c_double))
+            elif isinstance(m, GroupedAttention):
+                c.mixer, c.kv_heads, c.scale, c.chunk = 3, m.kv_heads, m.scale, m.chunk
+                c.kv_from = 0 if m.kv_from is None else m.kv_from + 1
+                c.rot_dim = c.rot_dims = m.rot.dims
+                c.rot_base, c.rot_divide = m.rot.base, m.rot.divide
+            elif isinstance(m, GatedLinearAttention):
+                c.mixer, c.gate_rank, c.tau = 4, m.rank, m.tau
         cc = _CStackConfig(mc.vocab_size, mc.hidden_size, len(mc.layers), layers, mc.loop_start, mc.loop_stop, mc.loop_times, mc.norm_eps,
-                           mc.logit_softcap, cfg.max_seq_len, cfg.max_batch, int(cfg.prefill_chunk_size or 0), int(cfg.dtype == "float32"))
+                           mc.logit_softcap, int(mc.design.post_norm), int(mc.design.silu), mc.embed_scale, int(mc.design.tied_head), cfg.max_seq_len, cfg.max_batch, int(cfg.prefill_chunk_size or 0), int(cfg.dtype == "float32"))
         model = C.c_void_p()
         check(lib().im_cuda_model_create_stack(engine._dev, C.byref(cc), C.byref(model)))
         return model
@@ -140,12 +157,9 @@ class LayerStack:
         check(lib().im_cuda_model_load_tensor(model, name.encode(), vp(data), C.c_int(dt), C.c_int(len(t.shape)), shape))
 
 
-# architecture names of the list-of-layers family; everything else is the quantized block family
-STACK_ARCHITECTURES = ("gizizen",)
-
-
 def family_of_name(architecture: str):
-    return LayerStack if architecture.lower() in STACK_ARCHITECTURES else QuantizedBlocks
+    """The designs of stack_config.py belong to the list-of-layers family; everything else is the quantized block family."""
+    return LayerStack if architecture.lower() in DESIGNS else QuantizedBlocks
 
 
 def family_of(config):

@@ -17,7 +17,8 @@ OBJ = os.path.join(HERE, "csrc", "_obj")
 LIB = os.path.join(HERE, "libironmill_cuda.so")
 # A library with one model family only: what a host that serves a single model has to compile.
 FAMILY_SOURCES = {
-    "stack": ("api.cu", "session.cu", "stack.cu", "dense.cu", "latent_attn.cu", "linear_attn.cu"),
+    "stack": ("api.cu", "session.cu", "stack.cu", "dense.cu", "latent_attn.cu", "grouped_attn.cu",
+              "linear_attn.cu", "linear_gated.cu"),
 }
 
 

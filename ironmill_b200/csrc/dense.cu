@@ -22,7 +22,11 @@ template <typename T>
 __device__ __forceinline__ void epi_pair(const DenseEpi &e, int m, int n, float v0, float v1, int N) {
     if (e.kind == kEpiProj) {
         if (n >= e.pair0) {
-            static_cast<T *>(e.act)[(size_t)m * e.ldact + ((n - e.pair0) >> 1)] = from_f<T>(gelu_tanh_f(v0) * v1);
+            static_cast<T *>(e.act)[(size_t)m * e.ldact + ((n - e.pair0) >> 1)] = from_f<T>((e.pair_silu ? silu_f(v0) : gelu_tanh_f(v0)) * v1);
+        } else if (n >= e.f0) {
+            float *f = e.xf + (size_t)m * e.ldx + (n - e.f0);
+            f[0] = v0;
+            if (n + 1 < N) f[1] = v1;
         } else {
             T *y = static_cast<T *>(e.y) + (size_t)m * e.ldy + n;
             if (n < e.silu_end) {
@@ -52,9 +56,10 @@ __device__ __forceinline__ void epi_pair(const DenseEpi &e, int m, int n, float 
     if (n + 1 < N) x[1] = v1;
 }
 
-// One row of the source as elements of type T (dst: K of them, then zeros up to ld), by the whole block.
+// One row of the source as elements of type T (dst: K of them, then zeros up to ld), by the whole block.  keep: this block
+// writes the row's new residual (kSrcAddNorm).
 template <typename T>
-__device__ __forceinline__ void stage_row(const DenseSrc &s, int m, int K, int ld, T *dst, float *sh) {
+__device__ __forceinline__ void stage_row(const DenseSrc &s, int m, int K, int ld, T *dst, float *sh, bool keep) {
     const int tid = threadIdx.x, nt = blockDim.x;
     if (s.kind == kSrcPlain) {
         constexpr int V = Vec16<T>::n;
@@ -71,6 +76,35 @@ __device__ __forceinline__ void stage_row(const DenseSrc &s, int m, int K, int l
         return;
     }
     float ss = 0.0f;
+    if (s.kind == kSrcAddNorm) {
+        const float *add = s.xf2 ? s.xf2 + (size_t)m * s.ldx : nullptr;
+        float inv = 0.0f;
+        if (add) {
+            for (int i = tid; i < K; i += nt) ss = fmaf(add[i], add[i], ss);
+            inv = 1.0f / sqrtf(block_sum_f(ss, sh) / (float)K + s.eps);
+        }
+        auto sum = [&](int i) { return add ? x[i] + add[i] * inv * s.gamma[i] : x[i]; };
+        float inv2 = 1.0f;
+        if (s.gamma2) {
+            ss = 0.0f;
+            for (int i = tid; i < K; i += nt) {
+                const float r = sum(i);
+                ss = fmaf(r, r, ss);
+            }
+            inv2 = 1.0f / sqrtf(block_sum_f(ss, sh) / (float)K + s.eps);
+        }
+        float *out = keep && s.xout ? s.xout + (size_t)m * s.ldx : nullptr;
+        for (int i = tid; i < ld; i += nt) {
+            float r = 0.0f;
+            if (i < K) {
+                r = sum(i);
+                if (out) out[i] = r;
+                if (s.gamma2) r *= inv2 * s.gamma2[i];
+            }
+            dst[i] = from_f<T>(r);
+        }
+        return;
+    }
     for (int i = tid; i < K; i += nt) ss = fmaf(x[i], x[i], ss);
     const float inv = 1.0f / sqrtf(block_sum_f(ss, sh) / (float)K + s.eps);
     for (int i = tid; i < ld; i += nt) dst[i] = from_f<T>(i < K ? x[i] * inv * s.gamma[i] : 0.0f);
@@ -106,7 +140,7 @@ __global__ void __launch_bounds__(kMvThreads, NB <= 4 ? 2 : 1) dense_matvec_kern
     pdl_trigger();
     load(blockIdx.x, 0);  // weights are constants: requested before the predecessor has finished
     pdl_wait();
-    for (int b = 0; b < B; b++) stage_row<T>(src, m0 + b, w.K, w.ld, xs + (size_t)b * w.ld, sh);
+    for (int b = 0; b < B; b++) stage_row<T>(src, m0 + b, w.K, w.ld, xs + (size_t)b * w.ld, sh, blockIdx.x == 0);
     __syncthreads();
     for (int tile = blockIdx.x; tile < ntiles; tile += gridDim.x) {
         const int n0 = (tile * groups + grp) * 2;
@@ -178,7 +212,7 @@ __global__ void __launch_bounds__(256) dense_stage_kernel(const DenseSrc src, in
     __shared__ float sh[32];
     pdl_trigger();
     pdl_wait();
-    stage_row<T>(src, blockIdx.x, K, ld, out + (size_t)blockIdx.x * ld, sh);
+    stage_row<T>(src, blockIdx.x, K, ld, out + (size_t)blockIdx.x * ld, sh, true);
 }
 
 // ---- tcgen05 GEMM ----------------------------------------------------------------------------------------------------
@@ -229,7 +263,8 @@ __device__ __forceinline__ void dense_tma_2d(void *dst, const CUtensorMap *map, 
 // bf16 epilogues: z sigmoid(z), and gelu_tanh(z) = z / (1 + exp(-2 u)), u = sqrt(2 / pi) (z + 0.044715 z^3); the error of the
 // fast exponential and quotient (about 1e-6) is far below the bf16 result's rounding
 __device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
-__device__ __forceinline__ float gelu_mul_fast(float z, float up) {
+__device__ __forceinline__ float pair_act_fast(float z, float up, bool silu) {
+    if (silu) return silu_fast(z) * up;
     const float w = -1.5957691216057308f * z * fmaf(0.044715f * z, z, 1.0f);
     return __fdividef(z * up, 1.0f + __expf(fminf(w, 80.0f)));
 }
@@ -265,21 +300,30 @@ __device__ __forceinline__ void dense_store16(const DenseGemm &p, int z, int n, 
             for (int i = 0; i < 16; i += 2) {
                 const float got = __shfl_xor_sync(0xffffffffu, odd ? v[i] : v[i + 1], 1);
                 if (pair) {
-                    const float r = odd ? gelu_mul_fast(got, v[i + 1]) : gelu_mul_fast(v[i], got);
+                    const float r = odd ? pair_act_fast(got, v[i + 1], e.pair_silu) : pair_act_fast(v[i], got, e.pair_silu);
                     if (n < p.N && i + odd < left) act[(size_t)(i + odd) * e.ldact] = from_f<T>(r);
                 } else {
 #pragma unroll
                     for (int j = 0; j < 2; j++)
-                        if (i + j < left) y[(size_t)(i + j) * e.ldy] = from_f<T>(n < e.silu_end ? silu_fast(v[i + j]) : v[i + j]);
+                        if (i + j < left) {
+                            if (n >= e.f0) e.xf[(size_t)(m + i + j) * e.ldx + (n - e.f0)] = v[i + j];
+                            else y[(size_t)(i + j) * e.ldy] = from_f<T>(n < e.silu_end ? silu_fast(v[i + j]) : v[i + j]);
+                        }
                 }
             }
         } else {
             T *y = static_cast<T *>(e.y) + (size_t)m * e.ldy + n;
             const bool act = n < e.silu_end;
-            if (n < p.N)
+            if (n < p.N && n >= e.f0) {
+                float *f = e.xf + (size_t)m * e.ldx + (n - e.f0);
+#pragma unroll
+                for (int i = 0; i < 16; i++)
+                    if (i < left) f[(size_t)i * e.ldx] = v[i];
+            } else if (n < p.N) {
 #pragma unroll
                 for (int i = 0; i < 16; i++)
                     if (i < left) y[(size_t)i * e.ldy] = from_f<T>(act ? silu_fast(v[i]) : v[i]);
+            }
         }
     } else if (n < p.N) {
         float *x = e.xf + (size_t)m * e.ldx + n;
@@ -462,21 +506,24 @@ __global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const DenseWeight w
 
 template <typename T>
 __global__ void __launch_bounds__(256) stack_embed_kernel(const uint32_t *__restrict__ tokens, const T *__restrict__ table, int ld, const float *__restrict__ gamma,
-                                                          float *__restrict__ x, float *__restrict__ x0, int W, uint32_t vocab, float eps) {
+                                                          float scale, float *__restrict__ x, float *__restrict__ x0, int W, uint32_t vocab, float eps) {
     __shared__ float sh[32];
     pdl_trigger();
     pdl_wait();
     const uint32_t tok = tokens[blockIdx.x];
     const T *row = table + (size_t)(tok < vocab ? tok : 0) * ld;
     const bool live = tok < vocab;
-    float ss = 0.0f;
-    for (int i = threadIdx.x; i < W; i += blockDim.x) {
-        const float v = live ? to_f<T>(row[i]) : 0.0f;
-        ss = fmaf(v, v, ss);
+    float ss = 0.0f, inv = scale;
+    if (gamma) {
+        for (int i = threadIdx.x; i < W; i += blockDim.x) {
+            const float v = live ? to_f<T>(row[i]) : 0.0f;
+            ss = fmaf(v, v, ss);
+        }
+        inv = 1.0f / sqrtf(block_sum_f(ss, sh) / (float)W + eps);
     }
-    const float inv = 1.0f / sqrtf(block_sum_f(ss, sh) / (float)W + eps);
     for (int i = threadIdx.x; i < W; i += blockDim.x) {
-        const float v = (live ? to_f<T>(row[i]) : 0.0f) * inv * gamma[i];
+        float v = (live ? to_f<T>(row[i]) : 0.0f) * inv;
+        if (gamma) v *= gamma[i];
         x[(size_t)blockIdx.x * W + i] = v;
         x0[(size_t)blockIdx.x * W + i] = v;
     }
@@ -617,13 +664,14 @@ int dense_project(const Device *dev, const DenseWeight &w, const DenseSrc &src, 
     return gemm_launch<32>(dev, p, w, x, ldx, slices, st);
 }
 
-int stack_embed(const uint32_t *tokens, const void *table, int f32, int ld, const float *gamma, float *x, float *x0, int width, uint32_t vocab, float eps, int M,
-                cudaStream_t st) {
+int stack_embed(const uint32_t *tokens, const void *table, int f32, int ld, const float *gamma, float scale, float *x, float *x0, int width, uint32_t vocab, float eps,
+                int M, cudaStream_t st) {
     if (M <= 0) return IM_OK;
-    if (f32) IM_CUDA_CHECK(launch_k(stack_embed_kernel<float>, dim3(M), dim3(256), 0, st, tokens, static_cast<const float *>(table), ld, gamma, x, x0, width, vocab, eps));
+    if (f32)
+        IM_CUDA_CHECK(launch_k(stack_embed_kernel<float>, dim3(M), dim3(256), 0, st, tokens, static_cast<const float *>(table), ld, gamma, scale, x, x0, width, vocab, eps));
     else
-        IM_CUDA_CHECK(launch_k(stack_embed_kernel<__nv_bfloat16>, dim3(M), dim3(256), 0, st, tokens, static_cast<const __nv_bfloat16 *>(table), ld, gamma, x, x0, width,
-                               vocab, eps));
+        IM_CUDA_CHECK(launch_k(stack_embed_kernel<__nv_bfloat16>, dim3(M), dim3(256), 0, st, tokens, static_cast<const __nv_bfloat16 *>(table), ld, gamma, scale, x, x0,
+                               width, vocab, eps));
     return IM_OK;
 }
 

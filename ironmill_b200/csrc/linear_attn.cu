@@ -5,6 +5,8 @@
 //                         S <- decay^n S + sum_j decay^(n-1-j) k_j v_j^T.  q, k, v are bf16 already; the f32 factors (state,
 //                         decayed scores, decayed values) enter a product as three bf16 terms each, which carry all 24 bits
 //   linear_finish_kernel  RMS norm over the heads together, sigmoid gate
+// The gated form has a decay per token and key channel in place of a constant per head, a norm per head and a SiLU gate; here it
+// runs token by token (everything in f32, short portions), linear_gated.cu has its decode step and its prompt chunks.
 // A sequence at position 0 starts from a zero state, whatever its slot held before.
 #include <algorithm>
 
@@ -17,25 +19,26 @@ namespace {
 constexpr int kLtCols = 32, kLtSlices = 8, kLtBlock = 8;  // value columns per CTA, shares of the key dimension, tokens staged at once
 
 // grid (heads, column blocks, sequences); warp = share of the key dimension, lane = value column.
-template <typename T, int DR>
+template <typename T, int DR, bool GATED>
 __global__ void __launch_bounds__(256) linear_step_kernel(const LinearArgs a) {
     extern __shared__ __align__(16) unsigned char linear_smem[];
     const LinearShape &s = a.s;
     float *qs = reinterpret_cast<float *>(linear_smem), *ks = qs + kLtBlock * s.dim, *vs = ks + kLtBlock * s.dim, *red = vs + kLtBlock * kLtCols;
+    float *as = red + kLtBlock * kLtSlices * kLtCols;  // gated: decays of the staged tokens
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int h = blockIdx.x, v0 = blockIdx.y * kLtCols, seq = blockIdx.z, col = v0 + lane;
     const bool live = col < s.vdim;
-    const float decay = a.pows[(size_t)h * (kLinearPow + 1) + 1];
+    const float decay = GATED ? 0.0f : a.pows[(size_t)h * (kLinearPow + 1) + 1];
     pdl_trigger();
     pdl_wait();
     const int slot = a.slot_map ? a.slot_map[seq] : seq;
-    float *state = a.state + ((size_t)slot * s.heads + h) * s.dim * s.vdim + col;
+    float *state = a.state + ((size_t)slot * s.heads + h) * s.dim * s.vS + col;
     const bool fresh = a.pos_dev[slot] == 0;
     float S[DR];
 #pragma unroll
     for (int i = 0; i < DR; i++) {
         const int d = i * kLtSlices + warp;
-        S[i] = (!fresh && live && d < s.dim) ? state[(size_t)d * s.vdim] : 0.0f;
+        S[i] = (!fresh && live && d < s.dim) ? state[(size_t)d * s.vS] : 0.0f;
     }
     for (int t0 = 0; t0 < a.T; t0 += kLtBlock) {
         const int nt = min(kLtBlock, a.T - t0);
@@ -43,7 +46,14 @@ __global__ void __launch_bounds__(256) linear_step_kernel(const LinearArgs a) {
         __syncthreads();
         for (int i = tid; i < nt * s.dim; i += 256) {
             const int b = i / s.dim, d = i % s.dim;
-            qs[i] = to_f<T>(y[(size_t)b * a.ldy + s.q_off + h * s.dimP + d]);
+            qs[i] = to_f<T>(y[(size_t)b * a.ldy + s.q_off + h * s.dimP + d]) * (GATED ? s.q_scale : 1.0f);
+            if (GATED) {
+                const int rank8 = (s.rank + 7) & ~7, HD = s.heads * s.dim;
+                const float *a1 = a.a1 + (size_t)(seq * a.T + t0 + b) * rank8, *a2 = a.a2 + h * s.dim + d;
+                float z = a.a2b[h * s.dim + d];
+                for (int r = 0; r < s.rank; r++) z = fmaf(a2[(size_t)r * HD], a1[r], z);
+                as[i] = expf(-softplus_f(-z) * s.inv_tau);
+            }
             ks[i] = to_f<T>(y[(size_t)b * a.ldy + s.k_off + h * s.dimP + d]);
         }
         for (int i = tid; i < nt * kLtCols; i += 256) {
@@ -58,7 +68,7 @@ __global__ void __launch_bounds__(256) linear_step_kernel(const LinearArgs a) {
             for (int i = 0; i < DR; i++) {
                 const int d = i * kLtSlices + warp;
                 if (d < s.dim) {
-                    S[i] = fmaf(decay, S[i], ks[b * s.dim + d] * v);
+                    S[i] = fmaf(GATED ? as[b * s.dim + d] : decay, S[i], ks[b * s.dim + d] * v);
                     o = fmaf(S[i], qs[b * s.dim + d], o);
                 }
             }
@@ -77,7 +87,7 @@ __global__ void __launch_bounds__(256) linear_step_kernel(const LinearArgs a) {
 #pragma unroll
         for (int i = 0; i < DR; i++) {
             const int d = i * kLtSlices + warp;
-            if (d < s.dim) state[(size_t)d * s.vdim] = S[i];
+            if (d < s.dim) state[(size_t)d * s.vS] = S[i];
         }
 }
 
@@ -91,7 +101,7 @@ inline size_t linear_chunk_smem(int C, int dimK, int bufs) {
 struct LinearSegments {
     int count = 1, tokens = 0;  // segments, tokens of each (a multiple of kLinearPow)
     int local = 0;
-    float *sums = nullptr;      // [count - 1][heads][dim][vdim]
+    float *sums = nullptr;      // [count - 1][heads][dim][vS]
 };
 
 // grid (column blocks of 32, heads, sequences or segments), C / 16 warps.  MW: 16-row tiles of the state per warp.
@@ -130,7 +140,7 @@ __global__ void __launch_bounds__(C * 2, 1) linear_chunk_kernel(const LinearArgs
     };
     load(0, t_begin);
     const int slot = a.slot_map ? a.slot_map[seq] : seq;
-    float *state = a.state + ((size_t)slot * s.heads + h) * s.dim * s.vdim + v0;
+    float *state = a.state + ((size_t)slot * s.heads + h) * s.dim * s.vS + v0;
     const bool fresh = a.pos_dev[slot] == 0 || sg.local;
     float S[MW][4][4];  // rows 16 mt + g (+ 8), columns 8 n + 2 t (+ 1); mt = warp + W * i
 #pragma unroll
@@ -140,14 +150,14 @@ __global__ void __launch_bounds__(C * 2, 1) linear_chunk_kernel(const LinearArgs
 #pragma unroll
             for (int e = 0; e < 4; e++) {
                 const int d = 16 * (warp + W * i) + g + 8 * (e >> 1), c = 8 * n + 2 * t + (e & 1);
-                S[i][n][e] = (!fresh && d < s.dim && v0 + c < s.vdim) ? state[(size_t)d * s.vdim + c] : 0.0f;
+                S[i][n][e] = (!fresh && d < s.dim && v0 + c < s.vdim) ? state[(size_t)d * s.vS + c] : 0.0f;
             }
     if (!sg.local && seg > 0) {
         const float d1 = a.pows[(size_t)h * (kLinearPow + 1) + kLinearPow];
         float dl = 1.0f;
         for (int i = 0; i < sg.tokens; i += kLinearPow) dl *= d1;
         for (int r = 0; r < seg; r++) {
-            const float *sum = sg.sums + ((size_t)r * s.heads + h) * s.dim * s.vdim + v0;
+            const float *sum = sg.sums + ((size_t)r * s.heads + h) * s.dim * s.vS + v0;
 #pragma unroll
             for (int i = 0; i < MW; i++)
 #pragma unroll
@@ -155,7 +165,7 @@ __global__ void __launch_bounds__(C * 2, 1) linear_chunk_kernel(const LinearArgs
 #pragma unroll
                     for (int e = 0; e < 4; e++) {
                         const int d = 16 * (warp + W * i) + g + 8 * (e >> 1), c = 8 * n + 2 * t + (e & 1);
-                        if (d < s.dim && v0 + c < s.vdim) S[i][n][e] = fmaf(S[i][n][e], dl, sum[(size_t)d * s.vdim + c]);
+                        if (d < s.dim && v0 + c < s.vdim) S[i][n][e] = fmaf(S[i][n][e], dl, sum[(size_t)d * s.vS + c]);
                     }
         }
     }
@@ -298,7 +308,7 @@ __global__ void __launch_bounds__(C * 2, 1) linear_chunk_kernel(const LinearArgs
         __syncthreads();
         if (bufs == 1 && ci + 1 < nchunks) load(0, c0 + C);
     }
-    float *out_state = sg.local ? sg.sums + ((size_t)seg * s.heads + h) * s.dim * s.vdim + v0 : state;
+    float *out_state = sg.local ? sg.sums + ((size_t)seg * s.heads + h) * s.dim * s.vS + v0 : state;
     if (sg.local || (!a.keep_state && seg == sg.count - 1))
 #pragma unroll
         for (int i = 0; i < MW; i++)
@@ -307,7 +317,7 @@ __global__ void __launch_bounds__(C * 2, 1) linear_chunk_kernel(const LinearArgs
 #pragma unroll
                 for (int e = 0; e < 4; e++) {
                     const int d = 16 * (warp + W * i) + g + 8 * (e >> 1), c = 8 * nb + 2 * t + (e & 1);
-                    if (d < s.dim && v0 + c < s.vdim) out_state[(size_t)d * s.vdim + c] = S[i][nb][e];
+                    if (d < s.dim && v0 + c < s.vdim) out_state[(size_t)d * s.vS + c] = S[i][nb][e];
                 }
 }
 
@@ -320,6 +330,18 @@ __global__ void __launch_bounds__(256) linear_finish_kernel(const LinearArgs a) 
     const int m = blockIdx.x, n = s.heads * s.vP;
     const float *o = a.o + (size_t)m * n;
     const T *gate = static_cast<const T *>(a.y) + (size_t)m * a.ldy + s.g_off;
+    if (s.gated) {  // a warp per head
+        T *out = static_cast<T *>(a.out) + (size_t)m * a.ldo;
+        for (int h = threadIdx.x >> 5; h < s.heads; h += 8) {
+            const float *oh = o + h * s.vP;
+            float ss = 0.0f;
+            for (int v = threadIdx.x & 31; v < s.vdim; v += 32) ss = fmaf(oh[v], oh[v], ss);
+            const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)s.vdim + s.eps);
+            for (int v = threadIdx.x & 31; v < s.vP; v += 32)
+                out[h * s.vP + v] = from_f<T>(v < s.vdim ? oh[v] * inv * a.norm[v] * silu_f(to_f<T>(gate[h * s.vP + v])) : 0.0f);
+        }
+        return;
+    }
     float ss = 0.0f;
     for (int i = threadIdx.x; i < n; i += 256)
         if (i % s.vP < s.vdim) ss = fmaf(o[i], o[i], ss);
@@ -332,8 +354,10 @@ constexpr size_t kLinearSmemMax = 226 * 1024;
 
 template <typename T, int DR>
 int step_launch(const LinearArgs &a, cudaStream_t st) {
-    const size_t smem = ((size_t)2 * kLtBlock * a.s.dim + kLtBlock * kLtCols + (size_t)kLtBlock * kLtSlices * kLtCols) * sizeof(float);
-    IM_CUDA_CHECK(launch_k(linear_step_kernel<T, DR>, dim3(a.s.heads, (a.s.vdim + kLtCols - 1) / kLtCols, a.nseq), dim3(256), smem, st, a));
+    const size_t smem = ((size_t)(a.s.gated ? 3 : 2) * kLtBlock * a.s.dim + kLtBlock * kLtCols + (size_t)kLtBlock * kLtSlices * kLtCols) * sizeof(float);
+    const dim3 grid(a.s.heads, (a.s.vdim + kLtCols - 1) / kLtCols, a.nseq);
+    if (a.s.gated) IM_CUDA_CHECK(launch_k(linear_step_kernel<T, DR, true>, grid, dim3(256), smem, st, a));
+    else IM_CUDA_CHECK(launch_k(linear_step_kernel<T, DR, false>, grid, dim3(256), smem, st, a));
     return IM_OK;
 }
 template <typename T>
@@ -368,18 +392,29 @@ int linear_prepare(const Device *dev) {
     static DeviceOnce once;
     if (!once.first(dev->ordinal)) return IM_OK;
 #define IM_SMEM(k) IM_CUDA_CHECK(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kLinearSmemMax))
-    IM_SMEM((linear_step_kernel<float, 64>)); IM_SMEM((linear_step_kernel<float, 32>));
-    IM_SMEM((linear_step_kernel<__nv_bfloat16, 64>)); IM_SMEM((linear_step_kernel<__nv_bfloat16, 32>));
+    IM_SMEM((linear_step_kernel<float, 64, false>)); IM_SMEM((linear_step_kernel<float, 32, false>));
+    IM_SMEM((linear_step_kernel<__nv_bfloat16, 64, false>)); IM_SMEM((linear_step_kernel<__nv_bfloat16, 32, false>));
+    IM_SMEM((linear_step_kernel<float, 64, true>)); IM_SMEM((linear_step_kernel<float, 32, true>));
+    IM_SMEM((linear_step_kernel<__nv_bfloat16, 64, true>)); IM_SMEM((linear_step_kernel<__nv_bfloat16, 32, true>));
     IM_SMEM((linear_chunk_kernel<128, 1>)); IM_SMEM((linear_chunk_kernel<64, 1>)); IM_SMEM((linear_chunk_kernel<64, 2>));
     IM_SMEM((linear_chunk_kernel<64, 4>));
 #undef IM_SMEM
-    return IM_OK;
+    return gated_prepare();
 }
 
 int linear_attention_run(const Device *dev, const LinearArgs &a, cudaStream_t st, int *launches) {
     const int dimK = round_up(a.s.dimP, 16), M = a.nseq * a.T;
     int rc = IM_ERR_BOUNDS;
-    if (!a.f32 && a.T >= 16 && dimK <= 256 && linear_chunk_smem(64, dimK, 1) <= kLinearSmemMax) {
+    if (a.s.gated) {
+        if (a.T == 1 && gated_decode_takes(a.s)) {
+            *launches += 1;
+            return gated_decode_run(a, st);
+        }
+        if (!a.f32 && a.nseq == 1 && a.T >= kGatedChunkMin && gated_chunk_takes(a.s)) {
+            rc = gated_chunk_run(a, st, launches);
+            if (rc != IM_ERR_BOUNDS) return rc;
+        }
+    } else if (!a.f32 && a.T >= 16 && dimK <= 256 && linear_chunk_smem(64, dimK, 1) <= kLinearSmemMax) {
         LinearSegments sg;
         sg.sums = a.seg_sums;
         const int ctas = (a.s.vdim + kLtCols - 1) / kLtCols * a.s.heads, per_sm = 2 * linear_chunk_smem(64, dimK, 1) <= kLinearSmemMax ? 2 : 1;

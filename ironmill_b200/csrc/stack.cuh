@@ -1,6 +1,7 @@
 // Building blocks of models described by a list of layers (stack.cu): dense bf16 / f32 projections with fused
-// prologues and epilogues (dense.cu), latent attention over a cache of latents (latent_attn.cu), decayed linear
-// attention with a recurrent state (linear_attn.cu).  Every block takes its sizes and constants as arguments.
+// prologues and epilogues (dense.cu), latent attention over a cache of latents (latent_attn.cu), grouped-query attention
+// over cached keys and values (grouped_attn.cu), decayed linear attention with a recurrent state (linear_attn.cu, and
+// linear_gated.cu for decays that depend on the token).  Every block takes its sizes and constants as arguments.
 //
 // Element type: `f32 == 0` keeps activations, weights and latent caches in bf16 (products accumulate in f32), `f32 == 1`
 // keeps all of them in f32 and never touches a reduced-precision unit.  The residual, norms, attention scores and
@@ -22,25 +23,30 @@ struct DenseWeight {
     void *w = nullptr;
 };
 
-// What the projection reads: activations as they are; rms(xf) * gamma; or the two f32 vectors [xf | xf2] side by side.
-enum { kSrcPlain = 0, kSrcNorm = 1, kSrcConcat = 2 };
+// What the projection reads: activations as they are; rms(xf) * gamma; the two f32 vectors [xf | xf2] side by side; or
+// r = xf + rms(xf2) * gamma (the residual with a sublayer's output normed and added), then rms(r) * gamma2 if gamma2 is there.
+// With xf2 == nullptr that is r = xf.  r goes to xout as well, if given (not the buffer xf).
+enum { kSrcPlain = 0, kSrcNorm = 1, kSrcConcat = 2, kSrcAddNorm = 3 };
 struct DenseSrc {
     int kind = kSrcPlain;
     const void *x = nullptr;      // kSrcPlain: elements [M, ldx]
     const float *xf = nullptr, *xf2 = nullptr;  // f32 [M, ldx]
-    const float *gamma = nullptr;
+    const float *gamma = nullptr, *gamma2 = nullptr;
+    float *xout = nullptr;
     int ldx = 0;
     int width = 0;                // columns of xf (and of xf2)
     float eps = 0.0f;
 };
 
-// Where it goes.  kEpiProj: rows below `pair0` to y (rows below `silu_end` through SiLU); rows from `pair0` on are
-// (gate, up) pairs, gelu_tanh(gate) * up to act.  kEpiResidual: xf[m, n] += sum.  kEpiF32: xf[m, n] = sum (+ bias[n]),
+// Where it goes.  kEpiProj: rows below `pair0` to y (rows below `silu_end` through SiLU), except that rows from `f0` on (a multiple
+// of eight) go to xf as f32, columns from 0; rows from `pair0` on are (gate, up) pairs, act(gate) * up to act, with gelu_tanh or
+// (pair_silu) SiLU.  kEpiResidual: xf[m, n] += sum.  kEpiF32: xf[m, n] = sum (+ bias[n]),
 // then cap * tanh(. / cap) when cap > 0.
 enum { kEpiProj = 0, kEpiResidual = 1, kEpiF32 = 2 };
 struct DenseEpi {
     int kind = kEpiProj;
-    int silu_end = 0, pair0 = 0;
+    int silu_end = 0, pair0 = 0, f0 = 1 << 30;
+    int pair_silu = 0;
     void *y = nullptr, *act = nullptr;
     float *xf = nullptr;
     const float *bias = nullptr;
@@ -57,9 +63,9 @@ int dense_project(const Device *dev, const DenseWeight &w, const DenseSrc &src, 
 int dense_prepare(const Device *dev);
 int dense_launches(int M, int K, int src_kind);
 
-// x[m] = x0[m] = rms(table[token]) * gamma (f32); tokens past the vocabulary read as zeros.
-int stack_embed(const uint32_t *tokens, const void *table, int f32, int ld, const float *gamma, float *x, float *x0, int width, uint32_t vocab, float eps, int M,
-                cudaStream_t st);
+// x[m] = x0[m] = rms(table[token]) * gamma, or without gamma table[token] * scale (f32); tokens past the vocabulary read as zeros.
+int stack_embed(const uint32_t *tokens, const void *table, int f32, int ld, const float *gamma, float scale, float *x, float *x0, int width, uint32_t vocab, float eps,
+                int M, cudaStream_t st);
 
 // ---- latent attention ------------------------------------------------------------------------------------------------
 // Per head a query [dim | rot_dim], a cached latent c (kv_rank, normed) and one rotated key part (rot_dim) shared by the
@@ -104,33 +110,87 @@ size_t latent_part_bytes(const Device *dev, const LatentShape &s, int tokens, in
 bool latent_expands(const LatentShape &s);  // prompt chunks of this shape can take the expanded form
 int latent_prepare(const Device *dev);
 
+// ---- grouped-query attention -------------------------------------------------------------------------------------------
+// q and k per head RMS-normed over dim (weights q_norm, k_norm) and rotated in their first rot_dims dimensions (neighbours
+// paired); a position sees its own chunk (chunk = 0: everything) up to itself; softmax with a keyless sink logit per head; heads
+// times sigmoid(gate).
+struct GroupedShape {
+    int heads, kv_heads, dim, vdim, rot_dims, chunk;
+    float scale, eps;
+    int dimP, vP;                    // per-head parts of the projected row and of a cache row, multiples of 8
+    int q_off, k_off, v_off, g_off;  // places in a projected row; k_off < 0: the cache belongs to another layer, which has filled it
+};
+void grouped_layout(GroupedShape *s, bool own_kv);
+
+struct GroupedArgs {
+    GroupedShape s;
+    int f32;
+    void *y;                 // projected rows [M, ldy]; queries may be normed and rotated in place
+    int ldy;
+    const float *q_norm, *k_norm;  // [dim]
+    const float *sink;       // [heads]
+    const float *cosc, *sinc;  // [max_seq, rot_dims / 2]
+    void *kcache, *vcache;   // [slots, kv_heads, max_seq, dimP], [slots, kv_heads, max_seq, vP]; padding is zero
+    int max_seq, nseq, T;
+    const int *pos_dev, *slot_map;
+    void *out;               // [M, ldo]: column h * vP
+    int ldo;
+    float *part;             // split partials scratch
+    size_t part_bytes;
+    unsigned *counters;      // [grouped_counters()], zero between launches
+    int host_pos, host_slot; // as in LatentArgs
+    int splits_ctx;
+};
+int grouped_attention_run(const Device *dev, const GroupedArgs &a, cudaStream_t st, int *launches);
+size_t grouped_part_bytes(const Device *dev, const GroupedShape &s, int f32, int tokens);
+int grouped_counters(const GroupedShape &s, int tokens);
+constexpr int kGroupedPrefillMin = 16;  // tokens of one sequence from which the prompt kernel runs (bf16)
+bool grouped_prefills(const GroupedShape &s);  // ... for shapes it takes
+int grouped_prepare(const Device *dev);
+
 // ---- decayed linear attention ----------------------------------------------------------------------------------------
 struct LinearShape {
     int heads, dim, vdim;
     int dimP, vP;
+    int vS;              // row stride of a state [dim, vS], a multiple of 4
     int q_off, k_off, v_off, g_off;
     float eps;
+    // gated form: a decay per token and key channel, sigmoid(a2 a1 + b)^(1 / tau); q scaled; norm over each head; SiLU gate
+    int gated, rank;
+    float inv_tau, q_scale;
 };
 struct LinearArgs {
     LinearShape s;
     int f32;
     const void *y;      // projected rows [M, ldy]: q | k | v (already activated) | gate
     int ldy;
-    const float *norm;  // [heads * vP], zeros in the padding
+    const float *norm;  // [heads * vP] (gated: [vP], shared by the heads), zeros in the padding
     const float *pows;  // [heads][kLinearPow + 1]: decay^0 .. decay^kLinearPow
-    float *state;       // [slots, heads, dim, vdim]
+    const float *a1;    // gated: f32 [M, rank8], rank8 = rank rounded up to 8
+    const float *a2, *a2b;  // gated: [rank, heads * dim] (transposed), [heads * dim]
+    float *decays;      // gated: [M, heads * dimP] f32 scratch of prompt chunks
+    float *chunk_states;  // gated: [chunks of kGatedChunk tokens][heads][dim][vS] f32 scratch (optional)
+    size_t chunk_bytes;
+    float *state;       // [slots, heads, dim, vS]
     int nseq, T;
     const int *pos_dev, *slot_map;
     int keep_state;     // 1: leave the state as it was (a pass that is not counted)
     float *o;           // [M, heads * vP] f32 scratch
-    float *seg_sums;    // [kLinearSegMax - 1][heads][dim][vdim] f32 scratch of a long prompt's segments (optional)
+    float *seg_sums;    // [kLinearSegMax - 1][heads][dim][vS] f32 scratch of a long prompt's segments (optional)
     void *out;          // [M, ldo]
     int ldo;
 };
 constexpr int kLinearPow = 128;
 constexpr int kLinearSegMax = 8;
+constexpr int kGatedChunk = 64, kGatedChunkMin = 16;  // tokens of a chunk; shortest portion that runs in chunks (bf16)
 int linear_attention_run(const Device *dev, const LinearArgs &a, cudaStream_t st, int *launches);
 int linear_prepare(const Device *dev);
+// linear_gated.cu, called by linear_attention_run: IM_ERR_BOUNDS when the shape or the scratch does not allow it
+bool gated_decode_takes(const LinearShape &s);
+bool gated_chunk_takes(const LinearShape &s);
+int gated_decode_run(const LinearArgs &a, cudaStream_t st);
+int gated_chunk_run(const LinearArgs &a, cudaStream_t st, int *launches);
+int gated_prepare();
 
 #ifdef __CUDACC__
 template <typename T>
@@ -183,6 +243,7 @@ struct Vec16<__nv_bfloat16> {
 
 __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float gelu_tanh_f(float z) {
     const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
     return 0.5f * z * (1.0f + tanhf(u));

@@ -124,6 +124,7 @@ class CudaInference:
             self._model = C.c_void_p()
         mc = provider.config()
         family = family_of(mc)
+        family.complete(mc, provider)
         self._mc, self._family = mc, family
         self._model = family.create(self, mc)
         if tq_signs is not None:
