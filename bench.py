@@ -24,6 +24,8 @@ shape; no checkpoint or dataset is read):
           the first two looped three times: eight layer passes) with random bf16 weights, beside a Llama-shaped model of
           this library with the same width, heads, feed-forward, vocabulary and number of passes (INT4 weights, fp16 KV):
           prefill of --prompt tokens and greedy decode at --batch; value = decode tok/s of the former.
+          --stack-design luvatar: the Luvatar design instead (eight layers: four of gated linear attention, four of
+          grouped-query attention, two of these on the keys of another), beside both Gizizen and the Llama-shaped model.
 
 `--impl reference` times the CPU restatement of the reference's own CPU path (the oracle) on the host
 cores for the same workload, on a bounded sample.
@@ -386,9 +388,17 @@ def run_decode(args, rank, world):
 STACK_SIZES = {"w2048": dict(width=2048, ff=8192, heads=16, vocab=32768), "w4096": dict(width=4096, ff=14336, heads=32, vocab=32768)}
 
 
-def stack_model_json(size):
+def stack_model_json(size, design="gizizen"):
+    """Eight layers (layer passes) of a design at a size."""
     z = STACK_SIZES[size]
     mlp = {"kind": "dense", "ff": z["ff"]}
+    if design == "luvatar":
+        gla = {"type": "gla", "mlp": mlp, "mixer": {"heads": z["heads"], "dim": 128, "vdim": 128, "tau": 16.0}}
+        mixer = {"heads": z["heads"], "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 8192},
+                 "rot": {"dims": 128, "base": 5e5, "scaling": {"factor": 4.0}}}
+        att, shared1, shared5 = ({"type": "attention", "mlp": mlp, "mixer": dict(mixer, **more)} for more in ({}, {"kv_from": 1}, {"kv_from": 5}))
+        return {"architecture": "Luvatar", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+                "layers": [gla, att, gla, shared1, gla, att, gla, shared5]}
     lat = {"type": "latent_attention", "mlp": mlp,
            "mixer": {"heads": z["heads"], "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5,
                      "rot": {"dims": 64, "base": 5e5, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}}
@@ -404,6 +414,7 @@ class SyntheticStackProvider:
     def __init__(self, obj, seed=77):
         from ironmill_b200.architectures import config_from_json
         self.cfg, self.seed = config_from_json(obj), seed
+        self.cfg.complete(lambda name: (16,))  # rank of the decays' gates
 
     def config(self):
         return self.cfg
@@ -419,14 +430,14 @@ class SyntheticStackProvider:
         from ironmill_b200.bundle import WeightTensor
         shape = self.cfg.tensors()[name]
         g = torch.Generator(device="cuda").manual_seed(self.seed * 7919 + zlib.crc32(name.encode()))
-        w = torch.ones(shape, device="cuda") if name.endswith(("norm", "norm1")) else torch.randn(shape, generator=g, device="cuda") * shape[-1] ** -0.5
+        w = torch.ones(shape, device="cuda") if name.endswith(("norm", "norm1", "norm2")) else torch.randn(shape, generator=g, device="cuda") * shape[-1] ** -0.5
         return WeightTensor(w.to(torch.bfloat16).view(torch.uint16).cpu().numpy(), shape, "bfloat16")
 
 
 def stack_flops_per_token(cfg, ctx):
     """Multiply-adds x 2 of one prompt token at mean context ctx: every projection, and attention in its expanded form
     (the expansion of a token's keys and values once)."""
-    from ironmill_b200.stack_config import LatentAttention
+    from ironmill_b200.stack_config import GroupedAttention, LatentAttention
     order = list(range(cfg.loop_start)) + list(range(cfg.loop_start, cfg.loop_stop)) * cfg.loop_times + list(range(cfg.loop_stop, len(cfg.layers)))
     w, n = cfg.hidden_size, 2 * cfg.hidden_size ** 2 * cfg.loop_times
     for i in order:
@@ -435,6 +446,8 @@ def stack_flops_per_token(cfg, ctx):
         n += 3 * w * L.ff + sum(a * b for a, b in (s for k, s in m.tensors(w).items() if len(s) == 2))
         if isinstance(m, LatentAttention):
             n += ctx * m.heads * (m.dim + m.rot_dim + m.vdim)
+        elif isinstance(m, GroupedAttention):
+            n += ctx * m.heads * (m.dim + m.vdim)
         else:
             n += 3 * m.heads * m.dim * m.vdim
     return 2 * n
@@ -477,13 +490,17 @@ def run_stack(args, rank, world):
     peak, peak_src = measured_peaks()
     tpeak = measured_tensor_peak()
     max_seq = P + W + K + 64
-    ours_p = SyntheticStackProvider(stack_model_json(args.stack_size))
-    cfg = ours_p.cfg
-    passes = len(cfg.layers) + (cfg.loop_stop - cfg.loop_start) * (cfg.loop_times - 1)
+    designs = {"stack": args.stack_design, "gizizen": "gizizen"}
+    passes = 8
     res, clocks = {}, None
-    which = ("stack", "blocks") if args.stack_arm == "both" else (args.stack_arm,)
+    which = (args.stack_arm,)
+    if args.stack_arm == "both":  # the design, and beside it the other families' models of the same size
+        which = ("stack", "blocks") if args.stack_design == "gizizen" else ("stack", "gizizen", "blocks")
     for arm in which:
-        if arm == "stack":
+        if arm in designs:
+            ours_p = SyntheticStackProvider(stack_model_json(args.stack_size, designs[arm]))
+            cfg = ours_p.cfg
+            assert len(cfg.layers) + (cfg.loop_stop - cfg.loop_start) * max(0, cfg.loop_times - 1) == passes
             eng = CudaInference(CudaConfig(max_seq_len=max_seq, max_batch=B))
             eng.load_weights(ours_p)
             flops = stack_flops_per_token(cfg, P / 2) * P
@@ -510,7 +527,7 @@ def run_stack(args, rank, world):
     print(json.dumps({
         "metric": "decode tok/s (list-of-layers model, bf16)", "value": first["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": K, "warmup": W,
         "ms_per_step": first["decode_ms_per_step"], "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
-        "config": dict(z, workload="stack", size=args.stack_size, layer_passes=passes, batch=B, prompt_tokens=P,
+        "config": dict(z, workload="stack", design=args.stack_design, size=args.stack_size, layer_passes=passes, batch=B, prompt_tokens=P,
                        l2_policy="inputs larger than L2: every step streams all weights"),
         "arms": res, "peaks": {"hbm_gbs": peak, "bf16_tflops": tpeak, "source": peak_src}, "clocks": clocks}))
 
@@ -926,7 +943,9 @@ def main():
     ap.add_argument("--kv-bits", type=int, default=8, choices=[4, 8, 16], help="attention workload: TurboQuant bits, or 16 = fp16 KV cache")
     ap.add_argument("--model", default="llama3_8b", choices=sorted(MODELS), help="decode workload shape (the default is the headline configuration)")
     ap.add_argument("--stack-size", default="w2048", choices=sorted(STACK_SIZES), help="stack workload: sizes of the model")
-    ap.add_argument("--stack-arm", default="both", choices=["both", "stack", "blocks"], help="stack workload: only the list-of-layers model, or only its Llama-shaped counterpart")
+    ap.add_argument("--stack-design", default="gizizen", choices=["gizizen", "luvatar"], help="stack workload: the design")
+    ap.add_argument("--stack-arm", default="both", choices=["both", "stack", "gizizen", "blocks"],
+                    help="stack workload: only the design, only Gizizen at that size, or only the Llama-shaped counterpart")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", 0))
     world = int(os.environ.get("WORLD_SIZE", 1))

@@ -50,3 +50,15 @@ def weights(cfg, seed=0, sharp=1.6):
             a = rng.normal(0, 1.0 / np.sqrt(shape[-1]), shape)
         out[name] = bf16(a)
     return out
+
+
+def close(got, want, dtype):
+    """For models of several layers.  Every sublayer's output is normed, so where one happens to be small its rounding is blown up:
+    rounding the plain model's activations to bf16 moves single rows of the tests' models by up to 0.11, all rows together by
+    less than 0.05.  So: all rows (eight and more) within TOL, and no row beyond three times that."""
+    got, want = np.asarray(got, dtype=np.float64), np.asarray(want)
+    d = got - want
+    d = d - d.mean(axis=-1, keepdims=True)
+    spread = np.sqrt(np.mean((want - want.mean(axis=-1, keepdims=True)) ** 2))
+    rows = np.sqrt((d * d).mean(axis=-1)) / spread
+    return rows.max() < 3 * TOL[dtype] and (len(rows) < 8 or np.sqrt((rows * rows).mean()) < TOL[dtype])

@@ -85,8 +85,8 @@ def test_mechanism(name, dtype):
     for n in (150, 40, 13):
         e.reset()
         got = e.prefill_all_logits(toks[:n])
-        assert L.error(got, want[:n]) < L.TOL[dtype]
-        assert L.error(decoded(e, toks[n:n + 12]), want[n:n + 12]) < L.TOL[dtype]
+        for rows, ref in ((got, want[:n]), (decoded(e, toks[n:n + 12]), want[n:n + 12])):
+            assert L.close(rows, ref, dtype) if name == "mix" else L.error(rows, ref) < L.TOL[dtype]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -102,7 +102,7 @@ def test_portions_of_every_size(dtype):
             rows.append(e.extend_sequence(sid, toks[at:at + n], range(n)))
             at += n
         assert e.sequence_position(sid) == 300
-        assert L.error(np.concatenate(rows), want) < L.TOL[dtype]
+        assert L.close(np.concatenate(rows), want, dtype)
         e.remove_sequence(sid)
 
 
@@ -116,9 +116,9 @@ def test_long_prompts_in_internal_chunks(dtype):
     for portion in (None, 300, 70, 5):
         e = engine(MIX, w, dtype, max_seq_len=700, prefill_chunk_size=portion)
         sid = e.open_sequence()
-        assert L.error(e.extend_sequence(sid, toks, places), want[places]) < L.TOL[dtype]
+        assert L.close(e.extend_sequence(sid, toks, places), want[places], dtype)
         e.reset()
-        assert L.error(e.prefill(toks)[None], want[-1:]) < L.TOL[dtype]
+        assert L.close(e.prefill(toks)[None], want[-1:], dtype)
         e.close()
 
 
@@ -235,9 +235,9 @@ def test_first_tokens(dtype):
     e = engine(MIX, w, dtype, max_seq_len=64)
     for n in range(1, 7):
         e.reset()
-        assert L.error(e.prefill(toks[:n])[None], want[n - 1:n]) < L.TOL[dtype]
+        assert L.close(e.prefill(toks[:n])[None], want[n - 1:n], dtype)
     e.reset()
-    assert L.error(decoded(e, toks), want) < L.TOL[dtype]
+    assert L.close(decoded(e, toks), want, dtype)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -254,20 +254,20 @@ def test_unequal_requests_in_a_batch(dtype, nseq):
     for k in range(4):
         for sid, lg in e.batch_decode_step({s: int(t[n + k]) for s, t, n in zip(ids, toks, lens)}):
             i = ids.index(sid)
-            assert L.error(lg[None], want[i][lens[i] + k:lens[i] + k + 1]) < L.TOL[dtype]
+            assert L.close(lg[None], want[i][lens[i] + k:lens[i] + k + 1], dtype)
     # one leaves, its slot goes to a new sequence; the rest decode on, in another order
     fresh = tokens(37, seed=999)
     fresh_want = OracleLuvatar(MIX, w).forward(fresh)
     e.remove_sequence(ids[0])
     sid = e.open_sequence()
     assert sid == ids[0]
-    assert L.error(e.extend_sequence(sid, fresh[:30], [29]), fresh_want[29:30]) < L.TOL[dtype]
+    assert L.close(e.extend_sequence(sid, fresh[:30], [29]), fresh_want[29:30], dtype)
     for k in range(4):
         feed = {sid: int(fresh[30 + k])}
         feed.update({ids[i]: int(toks[i][lens[i] + 4 + k]) for i in range(nseq - 1, 0, -1)})
         for s, lg in e.batch_decode_step(feed):
             ref = fresh_want[30 + k] if s == sid else want[ids.index(s)][lens[ids.index(s)] + 4 + k]
-            assert L.error(lg[None], ref[None]) < L.TOL[dtype]
+            assert L.close(lg[None], ref[None], dtype)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -282,7 +282,7 @@ def test_a_slot_used_again_remembers_nothing(dtype):
         e.remove_sequence(sid)
         sid = e.open_sequence()
         rows = [e.extend_sequence(sid, [int(t)], [0]) for t in b[:3]] + [e.extend_sequence(sid, b[3:], range(47))]
-        assert L.error(np.concatenate(rows), want) < L.TOL[dtype]
+        assert L.close(np.concatenate(rows), want, dtype)
         e.remove_sequence(sid)
 
 
@@ -293,7 +293,7 @@ def test_long_decoding(dtype):
     want = OracleLuvatar(MIX, w).forward(toks)
     e = engine(MIX, w, dtype, max_seq_len=420)
     e.prefill(toks[:5])
-    assert L.error(decoded(e, toks[5:]), want[5:]) < L.TOL[dtype]
+    assert L.close(decoded(e, toks[5:]), want[5:], dtype)
 
 
 @pytest.mark.parametrize("kv_heads", [1, 4])
@@ -374,11 +374,11 @@ def test_profiling_and_hidden_state_leave_the_sequence_alone():
     want = OracleLuvatar(MIX, w).forward(toks)
     e = engine(MIX, w, "float32", max_seq_len=64)
     e.prefill(toks[:20])
-    assert L.error((e.last_hidden_state() @ w["embed"].T.astype(np.float64))[None], want[19:20]) < L.TOL["float32"]
+    assert L.close((e.last_hidden_state() @ w["embed"].T.astype(np.float64))[None], want[19:20], "float32")
     assert e.profile_step()["attention"] > 0
     lg = decoded(e, toks[20:])
-    assert L.error(lg, want[20:]) < L.TOL["float32"]
-    assert L.error((e.last_hidden_state() @ w["embed"].T.astype(np.float64))[None], want[-1:]) < L.TOL["float32"]
+    assert L.close(lg, want[20:], "float32")
+    assert L.close((e.last_hidden_state() @ w["embed"].T.astype(np.float64))[None], want[-1:], "float32")
     assert e.step_launches() > 0 and e.step_bytes(30) > 0
 
 
@@ -399,14 +399,16 @@ def test_positions_and_going_back():
     e = engine(cfg, w, "float32", max_seq_len=64)
     e.prefill(np.concatenate([toks[:30], tokens(9, seed=7)]))
     e.truncate_to(30)
-    assert L.error(decoded(e, toks[30:]), want[30:]) < L.TOL["float32"]
+    assert L.close(decoded(e, toks[30:]), want[30:], "float32")
 
 
 def test_loading_is_checked():
     from ironmill_b200.engine import InferenceError
     cfg = L.config([L.attention(), L.gla()])
     w = L.weights(cfg, 26)
-    for name in ("l1.mix.norm", "l1.mix.a1", "l0.mix.k.norm", "l0.norm2", "final.norm"):
+    with pytest.raises(InferenceError, match="gate of rank"):
+        engine(cfg, {k: v for k, v in w.items() if k != "l1.mix.a1"}, "bfloat16", max_seq_len=16)
+    for name in ("l1.mix.norm", "l1.mix.a2", "l0.mix.k.norm", "l0.norm2", "final.norm"):
         with pytest.raises(InferenceError, match=name):
             engine(cfg, {k: v for k, v in w.items() if k != name}, "bfloat16", max_seq_len=16)
     for name in ("l0.mix.k", "l0.mix.q.norm", "l1.mix.a2", "l1.mix.a2.b"):
@@ -444,4 +446,4 @@ def test_trace_replay(tmp_path, dtype):
         assert f.exists() == bool(r)
         if r:
             got = np.fromfile(f, dtype="<f4").reshape(len(r), -1)
-            assert L.error(got, np.stack([want[k][p] for k, p in r])) < L.TOL[dtype]
+            assert L.close(got, np.stack([want[k][p] for k, p in r]), dtype)
