@@ -161,14 +161,18 @@ __global__ void __launch_bounds__(kGdWarps * 32) grouped_decode_kernel(const Gro
         *reinterpret_cast<uint4 *>(ring + i / (dimK / 8 - nk) * (rs + vs) + (nk + i % (dimK / 8 - nk)) * 16) = make_uint4(0, 0, 0, 0);
     for (int i = lane; i < kGdStages * kGdTile * (vK / 8 - nv); i += 32)
         *reinterpret_cast<uint4 *>(ring + i / (vK / 8 - nv) * (rs + vs) + rs + (nv + i % (vK / 8 - nv)) * 16) = make_uint4(0, 0, 0, 0);
+    // a lane copies the 16-byte vectors lc, lc + 32, ... of the rows lr, lr + rows, ... ([key | value] of a position is one row)
+    const int per = nk + nv, rows = per <= 32 ? 32 / per : 1, lr = per <= 32 ? lane / per : 0, lc = per <= 32 ? lane % per : lane;
     auto issue = [&](int it) {
-        if (it < ntiles) {
+        if (it < ntiles && lr < rows) {
             const int p0 = first + it * kGdUnit;
-            unsigned char *dst = ring + it % kGdStages * kGdTile * (rs + vs);
-            for (int i = lane; i < kGdTile * (nk + nv); i += 32) {
-                const int r = i / (nk + nv), c = i % (nk + nv), pp = min(p0 + r, r1 - 1);
-                if (c < nk) cp_async16(dst + r * (rs + vs) + c * 16, kc + (size_t)pp * s.dimP + c * 8);
-                else cp_async16(dst + r * (rs + vs) + rs + (c - nk) * 16, vc + (size_t)pp * s.vP + (c - nk) * 8);
+            unsigned char *dst = ring + it % kGdStages * kGdTile * (rs + vs) + lr * (rs + vs);
+            for (int c = lc; c < per; c += per <= 32 ? per : 32) {
+                const T *src = c < nk ? kc + c * 8 : vc + (c - nk) * 8;
+                const int stride = c < nk ? s.dimP : s.vP;
+                unsigned char *d = dst + (c < nk ? c * 16 : rs + (c - nk) * 16);
+#pragma unroll 4
+                for (int r = lr; r < kGdTile; r += rows, d += rows * (rs + vs)) cp_async16(d, src + (size_t)min(p0 + r, r1 - 1) * stride);
             }
         }
         cp_async_commit();

@@ -232,21 +232,31 @@ __global__ void __launch_bounds__(kGcThreads) gated_chunk_kernel(const LinearArg
         if (ib * 16 < n) {
             const int r0 = ib * 16 + g, cj = ib * 16 + 2 * t;  // rows r0, r0 + 8; columns cj, cj + 1 and 8 further on
             float acc[6] = {};
-            for (int d = 0; d < s.dim; d++) {
-                const float q0 = bf_at(qb + r0 * rs, d), q1 = bf_at(qb + (r0 + 8) * rs, d), e0 = bt[r0 * bs + d], e1 = bt[(r0 + 8) * bs + d];
-                float k[4], f[4];
+#pragma unroll 2
+            for (int d = 0; d < dimK; d += 2) {  // two channels; padding channels hold zeros
+                unsigned q[2], k[4];
+                float2 e[2], f[4];
+#pragma unroll
+                for (int j = 0; j < 2; j++) {
+                    q[j] = *reinterpret_cast<const unsigned *>(qb + (r0 + 8 * j) * rs + d * 2);
+                    e[j] = *reinterpret_cast<const float2 *>(bt + (r0 + 8 * j) * bs + d);
+                }
 #pragma unroll
                 for (int j = 0; j < 4; j++) {
                     const int c = cj + (j & 1) + 8 * (j >> 1);
-                    k[j] = bf_at(kb + c * rs, d);
-                    f[j] = bt[c * bs + d];
+                    k[j] = *reinterpret_cast<const unsigned *>(kb + c * rs + d * 2);
+                    f[j] = *reinterpret_cast<const float2 *>(bt + c * bs + d);
                 }
                 // the pairs above the diagonal, whose difference would be positive, are dropped below
+                auto add = [&](float &x, int r, int c) {
+                    x = fmaf(bf_lo(q[r]) * bf_lo(k[c]), exp2f(fminf(e[r].x - f[c].x, 0.0f)), x);
+                    x = fmaf(bf_hi(q[r]) * bf_hi(k[c]), exp2f(fminf(e[r].y - f[c].y, 0.0f)), x);
+                };
 #pragma unroll
                 for (int j = 0; j < 2; j++) {
-                    acc[j] = fmaf(q0 * k[j], exp2f(fminf(e0 - f[j], 0.0f)), acc[j]);
-                    acc[2 + j] = fmaf(q1 * k[j], exp2f(fminf(e1 - f[j], 0.0f)), acc[2 + j]);
-                    acc[4 + j] = fmaf(q1 * k[2 + j], exp2f(fminf(e1 - f[2 + j], 0.0f)), acc[4 + j]);
+                    add(acc[j], 0, j);
+                    add(acc[2 + j], 1, j);
+                    add(acc[4 + j], 1, 2 + j);
                 }
             }
             put(ib, ib, 0, 0, 2 * t <= g ? acc[0] : 0.0f, 2 * t + 1 <= g ? acc[1] : 0.0f);
